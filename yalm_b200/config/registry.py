@@ -15,6 +15,7 @@ from .llama import ConfigError, LlamaConfig
 from .nekotar import NekotarConfig
 from .rudazen import RudazenConfig
 from .samulorn import SamulornConfig
+from .saralix import SaralixConfig
 
 _ARCHITECTURES: Dict[str, Any] = {}
 
@@ -56,3 +57,4 @@ register_architecture("Golulix", GolulixConfig)
 register_architecture("Rudazen", RudazenConfig)
 register_architecture("Nekotar", NekotarConfig)
 register_architecture("Samulorn", SamulornConfig)
+register_architecture("Saralix", SaralixConfig)

@@ -304,7 +304,7 @@ int yalm_glu_clamp(const float* gu, int n_partials, long long partial_stride, vo
                    long long rows, int F, float alpha, float limit, float shift, int paired,
                    cudaStream_t stream);
 int yalm_routed_combine(float* x, const float* y, const int* pair_row, const float* weight,
-                        int n_tokens, int top, int dim, cudaStream_t stream);
+                        int n_tokens, int top, int dim, int accumulate, cudaStream_t stream);
 
 // ---- hyper.cu: several residual copies per token -----------------------------------------------
 // X [copies][rows][dim] float32.  Write (y not null): X_j <- sum_i mix[i][j] X_i + mult out_w[j] y, y the
@@ -329,18 +329,48 @@ int yalm_wkv_out(const float* o, const float* w, const float* gate, void* out, i
                  long long rows, int heads, int size, float eps, cudaStream_t stream);
 
 // ---- latent.cu: attention over a cached latent ---------------------------------------------------
-int yalm_latent_store(const float* dkv, int n_partials, long long partial_stride, const float* c_norm,
-                      float eps, const float* freq, const int* token_seq, const int* q_start,
-                      const int* seq_slot, const int* slot_pos, void* kv_step, void* cache, int dtype,
-                      int n_tokens, int rank, int rd, int hd, int capacity, int write_cache,
-                      const int* page_table, int pages_per_slot, int n_pages, cudaStream_t stream);
-int yalm_latent_absorb_q(const float* q, int n_partials, long long partial_stride, const void* w_uk,
-                         const float* freq, const int* token_seq, const int* q_start, const int* seq_slot,
-                         const int* slot_pos, void* q_out, int dtype, int n_tokens, int H, int dim, int rd,
-                         int rank, int hd, cudaStream_t stream);
-int yalm_latent_expand(const void* o, const void* w_uv, const float* gate, int n_partials,
-                       long long partial_stride, void* out, int dtype, int n_tokens, int H, int rank,
-                       int vdim, int hd, cudaStream_t stream);
+int yalm_latent_store(const float* src, int n_partials, long long partial_stride, int src_row, int col0,
+                      const float* c_norm, float eps, const float* freq, int halves, float mult,
+                      const int* token_seq, const int* q_start, const int* seq_slot, const int* slot_pos,
+                      void* kv_step, void* cache, void* c_rows, int dtype, int n_tokens, int rank, int rd,
+                      int hd, int capacity, int write_cache, const int* page_table, int pages_per_slot,
+                      int n_pages, cudaStream_t stream);
+int yalm_latent_rotate_q(const float* q, int n_partials, long long partial_stride, int q_row, int col0,
+                         const float* freq, int halves, float mult, const int* token_seq,
+                         const int* q_start, const int* seq_slot, const int* slot_pos, void* q_out,
+                         int dtype, int n_tokens, int H, int dim, int rd, cudaStream_t stream);
+int yalm_latent_absorb_q(const float* q, int n_partials, long long partial_stride, int q_row, int col0,
+                         const void* w_uk, const float* freq, int halves, float mult, const int* token_seq,
+                         const int* q_start, const int* seq_slot, const int* slot_pos, void* q_out,
+                         int dtype, int n_tokens, int H, int dim, int rd, int rank, int hd,
+                         cudaStream_t stream);
+int yalm_latent_expand(const void* o, const float* part_o, const float* part_ml, int nsplit,
+                       const void* w_uv, const float* gate, int gate_mode, int n_partials,
+                       long long partial_stride, int gate_row, int col0, void* out, int dtype, int n_tokens,
+                       int H, int rank, int vdim, int hd, cudaStream_t stream);
+
+// ---- latent_attention.cu -------------------------------------------------------------------------
+int yalm_latent_attention_mma_usable(int dtype, int rank, int hd);
+int yalm_latent_attention(const void* q, const void* kv_step, const void* cache, const int* token_seq,
+                          const int* q_start, const int* seq_slot, const int* slot_pos, void* out,
+                          float* part_o, float* part_ml, int dtype, int n_tokens, int H, int rank, int hd,
+                          int capacity, int window, float scale, const float* sink, int nsplit, int mma,
+                          const int* page_table, int pages_per_slot, int n_pages, cudaStream_t stream);
+int yalm_latent_prefill_usable(int dtype, int dim, int rd, int vdim, int rank, int hd);
+int yalm_latent_prefill(const void* q, const void* kv, const void* kv_step, const int* q_start, void* out,
+                        int dtype, int n_seqs, int max_q_len, int H, int dim, int rd, int vdim, int rank,
+                        int hd, int window, float scale, const float* sink, const float* gate,
+                        int gate_mode, int gate_n, long long gate_stride, int gate_row, int gate_col0,
+                        cudaStream_t stream);
+
+// ---- ssd.cu: a state-space recurrence with one decay per head ------------------------------------
+int yalm_ssd_scan(const float* act, const float* dt, int dt_n, long long dt_stride, int dt_row, int col0,
+                  const float* dt_bias, const float* a_log, const float* d_skip, const int* q_start,
+                  const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int G,
+                  int P, int N, cudaStream_t stream);
+int yalm_gated_group_norm(const float* y, const float* z, int z_n, long long z_stride, int z_row, int col0,
+                          const float* w, void* out, int out_dtype, int rows, int inner, int groups,
+                          float eps, cudaStream_t stream);
 
 // ---- small_ops.cu ---------------------------------------------------------------------------------
 // out [n] = act(sum of n_partials slices of z [n]): act 1 = gelu (tanh form), 2 = tanh

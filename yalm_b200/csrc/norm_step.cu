@@ -7,6 +7,8 @@
 //    where post and pre are each one of
 //        tanh form ("dynamic tanh"):  n(v) = tanh(alpha v) w + b       no mean, no variance
 //        rms form:                    n(v) = v / sqrt(mean(v^2) + eps) w
+//        layer form:                  n(v) = (v - mean v) / sqrt(mean((v - mean v)^2) + eps) w
+//                                     (two passes over the row: the deviations are squared, not v)
 //        none:                        post: x <- x + y;  pre: h = x in the storage type
 //    or absent.  With a row list the kernel only reads: h[r] = pre(x[rows[r]]).
 //  * short_conv: a causal convolution over time on every channel of a product's output,
@@ -22,7 +24,7 @@
 namespace yalm {
 
 struct NormForm {
-  int kind;              // 0 absent, 1 tanh form, 2 rms form, 3 none (plain add / plain cast)
+  int kind;              // 0 absent, 1 tanh form, 2 rms form, 3 none (plain add / plain cast), 4 layer form
   const float* w;
   const float* b;        // tanh form only
   float alpha, eps;
@@ -64,6 +66,19 @@ __device__ __forceinline__ void store4(T* __restrict__ p, float a, float b, floa
   }
 }
 
+// this thread's part of sum((row - mean)^2); every thread reads the elements it wrote itself
+template <int W>
+__device__ __forceinline__ float row_deviations(const float* row, float mean, int i0, int step, int dim) {
+  float ss = 0.f;
+  for (int i = i0; i < dim; i += step)
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      const float d = row[i + j] - mean;
+      ss += d * d;
+    }
+  return ss;
+}
+
 // VEC: dim is a multiple of four and every pointer 16-byte aligned: a thread takes four neighbouring features
 template <typename T, bool VEC>
 __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, NormForm post, NormForm pre,
@@ -76,6 +91,7 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
   float* xr = x + t * dim;
   constexpr int W = VEC ? 4 : 1;
   const int i0 = threadIdx.x * W, step = blockDim.x * W;
+  float sum = 0.f;                                         // this thread's part of the row that is read
   if (post.kind) {
     float ss = 0.f;
     for (int i = i0; i < dim; i += step) {
@@ -92,10 +108,15 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
         if (B.p != nullptr) y[0] = fmaf(B.factor, sum_slices(B.p + t * dim + i, B.n, B.stride), y[0]);
       }
 #pragma unroll
-      for (int j = 0; j < W; ++j) { row_s[i + j] = y[j]; ss += y[j] * y[j]; }
+      for (int j = 0; j < W; ++j) { row_s[i + j] = y[j]; ss += post.kind == 4 ? y[j] : y[j] * y[j]; }
     }
-    float r = 1.f;
+    float r = 1.f, mean = 0.f;
     if (post.kind == 2) r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dim + post.eps);
+    if (post.kind == 4) {
+      mean = block_sum(ss, scratch) / (float)dim;
+      r = 1.0f / sqrtf(block_sum(row_deviations<W>(row_s, mean, i0, step, dim), scratch) / (float)dim + post.eps);
+    }
+    float vs = 0.f;                                        // the new x's sum, for a layer-form read
     for (int i = i0; i < dim; i += step) {
       float v[W];
       if constexpr (VEC) {
@@ -109,21 +130,30 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
         const float y = row_s[i + j];
         if (post.kind == 1) v[j] += apply_tanh_form(post, y, i + j);
         else if (post.kind == 2) v[j] += y * r * post.w[i + j];
+        else if (post.kind == 4) v[j] += (y - mean) * r * post.w[i + j];
         else v[j] += y;
         row_s[i + j] = v[j];
+        vs += v[j];
       }
       if constexpr (VEC) *reinterpret_cast<float4*>(xr + i) = make_float4(v[0], v[1], v[2], v[3]);
       else xr[i] = v[0];
     }
+    sum = vs;
   } else if (pre.kind) {
     for (int i = i0; i < dim; i += step) {
       if constexpr (VEC) *reinterpret_cast<float4*>(row_s + i) = *reinterpret_cast<const float4*>(xr + i);
       else row_s[i] = xr[i];
+#pragma unroll
+      for (int j = 0; j < W; ++j) sum += row_s[i + j];
     }
   }
   if (!pre.kind) return;
   T* out = h + (size_t)blockIdx.x * dim;
-  float r = 1.f;
+  float r = 1.f, mean = 0.f;
+  if (pre.kind == 4) {
+    mean = block_sum(sum, scratch) / (float)dim;
+    r = 1.0f / sqrtf(block_sum(row_deviations<W>(row_s, mean, i0, step, dim), scratch) / (float)dim + pre.eps);
+  }
   if (pre.kind == 2) {
     float ss = 0.f;
     for (int i = i0; i < dim; i += step)
@@ -136,7 +166,8 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
 #pragma unroll
     for (int j = 0; j < W; ++j) {
       const float v = row_s[i + j];
-      o[j] = pre.kind == 2 ? v * r * pre.w[i + j] : (pre.kind == 1 ? apply_tanh_form(pre, v, i + j) : v);
+      o[j] = pre.kind == 4 ? (v - mean) * r * pre.w[i + j]
+           : pre.kind == 2 ? v * r * pre.w[i + j] : (pre.kind == 1 ? apply_tanh_form(pre, v, i + j) : v);
     }
     if constexpr (VEC) store4<T>(out + i, o[0], o[1], o[2], o[3]);
     else out[i] = from_float<T>(o[0]);
@@ -275,7 +306,7 @@ using namespace yalm;
 
 // x float32 [.., dim] (changed in place when post_kind != 0).  y = fa * sum(slices a) + fb * sum(slices b)
 // (either may be null).  post / pre: kind 0 absent, 1 tanh form (w, b, alpha), 2 rms form (w, eps),
-// 3 none.  h [n_rows][dim] in h_dtype receives pre(x).  rows (optional, only without a post step): the
+// 3 none, 4 layer form (w, eps).  h [n_rows][dim] in h_dtype receives pre(x).  rows (optional, only without a post step): the
 // rows of x that are read.
 extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, float fa, const float* b,
                               int nb, long long sb, float fb, int post_kind, const float* post_w,

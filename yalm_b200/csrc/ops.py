@@ -94,7 +94,7 @@ _SIGNATURES = {
     "yalm_gemm_2sm_act": [_vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     "yalm_gemm_grouped_tc": [_vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _f, _f,
                              _f, _vp, _vp],
-    "yalm_routed_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "yalm_routed_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "yalm_attention_pooled": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
                               _i, _i, _f, _i, _vp, _i, _i, _vp, _vp, _i, _i, _vp, _i, _i, _vp],
     "yalm_attention_exact_prefill": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i,
@@ -115,10 +115,20 @@ _SIGNATURES = {
     "yalm_wkv": [_vp, _i, _ll, _vp, _i, _ll, _vp, _i, _ll, _vp, _i, _ll, _vp, _i, _ll, _vp, _vp, _vp, _vp,
                  _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "yalm_wkv_out": [_vp, _vp, _vp, _vp, _i, _ll, _i, _i, _f, _vp],
-    "yalm_latent_store": [_vp, _i, _ll, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                          _i, _vp, _i, _i, _vp],
-    "yalm_latent_absorb_q": [_vp, _i, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "yalm_latent_expand": [_vp, _vp, _vp, _i, _ll, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "yalm_latent_store": [_vp, _i, _ll, _i, _i, _vp, _f, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i,
+                          _i, _i, _i, _i, _vp, _i, _i, _vp],
+    "yalm_latent_rotate_q": [_vp, _i, _ll, _i, _i, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "yalm_latent_absorb_q": [_vp, _i, _ll, _i, _i, _vp, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
+                             _i, _vp],
+    "yalm_latent_expand": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _ll, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "yalm_latent_attention_mma_usable": [_i, _i, _i],
+    "yalm_latent_attention": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp,
+                              _i, _i, _vp, _i, _i, _vp],
+    "yalm_latent_prefill_usable": [_i, _i, _i, _i, _i, _i],
+    "yalm_latent_prefill": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _ll,
+                            _i, _i, _vp],
+    "yalm_ssd_scan": [_vp, _vp, _i, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "yalm_gated_group_norm": [_vp, _vp, _i, _ll, _i, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "yalm_activation_rows": [_vp, _i, _ll, _vp, _i, _ll, _i, _vp],
     "yalm_norm_step": [_vp, _vp, _i, _ll, _f, _vp, _i, _ll, _f, _i, _vp, _vp, _f, _f, _i, _vp, _vp, _f, _f, _vp,
                        _i, _vp, _i, _i, _vp],
@@ -967,50 +977,182 @@ def wkv_out(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, out: torc
 
 
 # ---- attention over a cached latent ----------------------------------------------------------------
-def latent_store(dkv: torch.Tensor, n_partials: int, c_norm: torch.Tensor, eps: float, freq: torch.Tensor,
+GATE_NONE, GATE_HEAD, GATE_ELEMENT = 0, 1, 2
+
+
+def _columns(src: torch.Tensor, n_partials: int, n: int, col0: int, width: int, what: str):
+    """(pointer, slices, slice stride, row pitch, first column) of ``width`` columns of a stacked product,
+    float32 slices [(s,) n, row]."""
+    row = src.shape[-1]
+    _need(src.dtype == torch.float32 and src.is_contiguous() and src.shape[-2] == n and col0 + width <= row
+          and src.numel() >= n_partials * n * row, what)
+    return _p(src), int(n_partials), n * row, row, int(col0)
+
+
+def latent_store(src: torch.Tensor, n_partials: int, c_norm: torch.Tensor, eps: float, freq: torch.Tensor,
                  batch, slot_pos: torch.Tensor, kv_step: torch.Tensor, cache: torch.Tensor, rank: int,
-                 rd: int, hd: int, capacity: int, write_cache: bool = True, pages=None) -> None:
-    """dkv float32 [(s,) N, rank + rd] -> the row [norm(c) w | rot(kr) | 0] of every token, to
-    kv_step [N, 2, 1, hd] (key and value alike) and to the cache."""
+                 rd: int, hd: int, capacity: int, write_cache: bool = True, pages=None, col0: int = 0,
+                 halves: bool = False, mult: float = 1.0, c_rows: Optional[torch.Tensor] = None) -> None:
+    """The rank + rd columns from ``col0`` of src float32 [(s,) N, row] -> the row [norm(c) w | rot(kr) | 0]
+    of every token, to kv_step [N, 2, 1, hd] (key and value alike) and to the cache (of a step longer than
+    a ring the rows that the ring keeps); ``c_rows`` [N, rank] (optional) receives norm(c) w alone.  The
+    rotation turns pairs (2i, 2i + 1), or (i, i + rd/2) with ``halves``; cos and sin times ``mult``."""
     n = kv_step.shape[0]
     pt, pps, npg = _pages(pages, cache, 1, hd)
-    _need(dkv.dtype == torch.float32 and dkv.is_contiguous() and dkv.shape[-1] == rank + rd
-          and dkv.shape[-2] == n and c_norm.dtype == freq.dtype == torch.float32 and c_norm.numel() == rank
+    _need(c_norm.dtype == freq.dtype == torch.float32 and c_norm.numel() == rank
           and freq.numel() >= max(1, rd // 2) and kv_step.dtype == cache.dtype and kv_step.is_contiguous()
           and kv_step.numel() == n * 2 * hd and cache.is_contiguous(), "latent_store: shapes")
-    _check(lib().yalm_latent_store(_p(dkv), n_partials, n * (rank + rd), _p(c_norm), float(eps), _p(freq),
+    _need(c_rows is None or (c_rows.dtype == cache.dtype and c_rows.is_contiguous() and c_rows.numel() == n * rank),
+          "latent_store: c_rows [N, rank]")
+    _check(lib().yalm_latent_store(*_columns(src, n_partials, n, col0, rank + rd, "latent_store: source columns"),
+                                   _p(c_norm), float(eps), _p(freq), 1 if halves else 0, float(mult),
                                    _p(batch.token_seq), _p(batch.q_start), _p(batch.seq_slot), _p(slot_pos),
-                                   _p(kv_step), _p(cache), dtype_code(cache.dtype), n, rank, rd, hd, capacity,
-                                   1 if write_cache else 0, pt, pps, npg, _stream()), "latent_store")
+                                   _p(kv_step), _p(cache), _p(c_rows), dtype_code(cache.dtype), n, rank, rd, hd,
+                                   capacity, 1 if write_cache else 0, pt, pps, npg, _stream()), "latent_store")
+
+
+def latent_rotate_q(q: torch.Tensor, n_partials: int, freq: torch.Tensor, batch, slot_pos: torch.Tensor,
+                    q_out: torch.Tensor, H: int, dim: int, rd: int, col0: int = 0, halves: bool = False,
+                    mult: float = 1.0) -> None:
+    """q_out [N, H, dim + rd] = the columns from ``col0`` of q float32 [(s,) N, row] with the last rd features
+    of every head rotated, in q_out's type."""
+    n = batch.n_tokens
+    _need(q_out.is_contiguous() and q_out.numel() == n * H * (dim + rd) and freq.dtype == torch.float32
+          and freq.numel() >= max(1, rd // 2), "latent_rotate_q: shapes")
+    _check(lib().yalm_latent_rotate_q(*_columns(q, n_partials, n, col0, H * (dim + rd), "latent_rotate_q: source columns"),
+                                      _p(freq), 1 if halves else 0, float(mult), _p(batch.token_seq),
+                                      _p(batch.q_start), _p(batch.seq_slot), _p(slot_pos), _p(q_out),
+                                      dtype_code(q_out.dtype), n, H, dim, rd, _stream()), "latent_rotate_q")
 
 
 def latent_absorb_q(q: torch.Tensor, n_partials: int, w_uk: torch.Tensor, freq: torch.Tensor, batch,
                     slot_pos: torch.Tensor, q_out: torch.Tensor, H: int, dim: int, rd: int, rank: int,
-                    hd: int) -> None:
-    """q float32 [(s,) N, H (dim + rd)], w_uk [H, dim, rank] -> q_out [N, H, hd] =
+                    hd: int, col0: int = 0, halves: bool = False, mult: float = 1.0) -> None:
+    """The columns from ``col0`` of q float32 [(s,) N, row], w_uk [H, dim, rank] -> q_out [N, H, hd] =
     [Wuk_h^T q_h[:dim] | rot(q_h[dim:]) | 0]."""
     n = q_out.shape[0]
-    _need(q.dtype == torch.float32 and q.is_contiguous() and q.shape[-1] == H * (dim + rd) and q.shape[-2] == n
-          and w_uk.dtype == q_out.dtype and w_uk.is_contiguous() and w_uk.numel() == H * dim * rank
+    _need(w_uk.dtype == q_out.dtype and w_uk.is_contiguous() and w_uk.numel() == H * dim * rank
           and q_out.is_contiguous() and q_out.numel() == n * H * hd and freq.dtype == torch.float32,
           "latent_absorb_q: shapes")
-    _check(lib().yalm_latent_absorb_q(_p(q), n_partials, n * H * (dim + rd), _p(w_uk), _p(freq),
-                                      _p(batch.token_seq), _p(batch.q_start), _p(batch.seq_slot), _p(slot_pos),
-                                      _p(q_out), dtype_code(q_out.dtype), n, H, dim, rd, rank, hd, _stream()),
+    _check(lib().yalm_latent_absorb_q(*_columns(q, n_partials, n, col0, H * (dim + rd), "latent_absorb_q: source columns"),
+                                      _p(w_uk), _p(freq), 1 if halves else 0, float(mult), _p(batch.token_seq),
+                                      _p(batch.q_start), _p(batch.seq_slot), _p(slot_pos), _p(q_out),
+                                      dtype_code(q_out.dtype), n, H, dim, rd, rank, hd, _stream()),
            "latent_absorb_q")
 
 
-def latent_expand(o: torch.Tensor, w_uv: torch.Tensor, gate: Optional[torch.Tensor], n_partials: int,
-                  out: torch.Tensor, H: int, rank: int, vdim: int, hd: int) -> None:
-    """o [N, H, hd], w_uv [H, rank, vdim] -> out [N, H vdim] = (Wuv_h o_h[:rank]) sigmoid(gate)."""
+def latent_expand(o: Optional[torch.Tensor], w_uv: torch.Tensor, gate: Optional[torch.Tensor], n_partials: int,
+                  out: torch.Tensor, H: int, rank: int, vdim: int, hd: int, parts=None, gate_col0: int = 0,
+                  gate_mode: int = GATE_ELEMENT) -> None:
+    """o [N, H, hd] (or ``parts`` = (part_o, part_ml, nsplit) of a split attention, merged here), w_uv
+    [H, rank, vdim] -> out [N, H vdim] = (Wuv_h o_h[:rank]) sigmoid(gate); the gate's logits are columns
+    from ``gate_col0`` of float32 slices [(s,) N, row], one per feature or (GATE_HEAD) one per head."""
     n = out.shape[0]
-    _need(o.dtype == w_uv.dtype == out.dtype and o.is_contiguous() and o.numel() == n * H * hd
-          and w_uv.is_contiguous() and w_uv.numel() == H * rank * vdim and out.is_contiguous()
-          and out.shape[1] == H * vdim, "latent_expand: shapes")
-    _need(gate is None or (gate.dtype == torch.float32 and gate.is_contiguous()
-                           and gate.numel() >= n_partials * n * H * vdim), "latent_expand: gate slices")
-    _check(lib().yalm_latent_expand(_p(o), _p(w_uv), _p(gate), n_partials, n * H * vdim, _p(out),
-                                    dtype_code(out.dtype), n, H, rank, vdim, hd, _stream()), "latent_expand")
+    _need(w_uv.dtype == out.dtype and w_uv.is_contiguous() and w_uv.numel() == H * rank * vdim
+          and out.is_contiguous() and out.shape[1] == H * vdim, "latent_expand: shapes")
+    part_o, part_ml, nsplit = parts if parts is not None else (None, None, 1)
+    if nsplit > 1:
+        _need(part_o.dtype == part_ml.dtype == torch.float32 and part_o.numel() >= n * H * nsplit * rank
+              and part_ml.numel() >= n * H * nsplit * 2, "latent_expand: partial results")
+    else:
+        _need(o is not None and o.dtype == out.dtype and o.is_contiguous() and o.numel() == n * H * hd,
+              "latent_expand: o [N, H, hd]")
+    g = (None, 0, 0, 0, 0)
+    if gate is not None:
+        g = _columns(gate, n_partials, n, gate_col0, H if gate_mode == GATE_HEAD else H * vdim, "latent_expand: gate slices")
+    _check(lib().yalm_latent_expand(_p(o), _p(part_o), _p(part_ml), int(nsplit), _p(w_uv), g[0], int(gate_mode), *g[1:],
+                                    _p(out), dtype_code(out.dtype), n, H, rank, vdim, hd, _stream()), "latent_expand")
+
+
+LATENT_MAX_SPLIT = 64
+LATENT_FEW_TOKENS = 128          # the most tokens whose split results latent_expand merges
+
+
+def latent_attention_mma_usable(dtype: torch.dtype, rank: int, hd: int) -> bool:
+    return dtype in HALF_TYPES and bool(lib().yalm_latent_attention_mma_usable(dtype_code(dtype), rank, hd))
+
+
+def latent_attention(q: torch.Tensor, kv_step: torch.Tensor, cache: torch.Tensor, batch, slot_pos: torch.Tensor,
+                     out: Optional[torch.Tensor], H: int, rank: int, hd: int, capacity: int, window: Optional[int],
+                     scale: float, sink: Optional[torch.Tensor] = None, pages=None, parts=None,
+                     mma: bool = True) -> None:
+    """The absorbed form: every query q [N, H, hd] over the latent rows it sees (positions of this step from
+    kv_step [N, 2, 1, hd], earlier ones from the cache), the last ``window`` positions or all; ``sink``
+    float32 [H] adds exp(sink_h) to the denominator.  out [N, H, hd] (its first ``rank`` features), or with
+    ``parts`` = (part_o, part_ml, nsplit) the results of nsplit runs of keys for ``latent_expand``."""
+    n = batch.n_tokens
+    pt, pps, npg = _pages(pages, cache, 1, hd)
+    part_o, part_ml, nsplit = parts if parts is not None else (None, None, 1)
+    _need(q.dtype == kv_step.dtype == cache.dtype and q.is_contiguous() and q.numel() == n * H * hd
+          and kv_step.is_contiguous() and kv_step.numel() == n * 2 * hd and cache.is_contiguous(),
+          "latent_attention: shapes")
+    _need(nsplit > 1 or (out is not None and out.dtype == q.dtype and out.is_contiguous()
+                         and out.numel() == n * H * hd), "latent_attention: out [N, H, hd]")
+    _need(nsplit == 1 or (part_o.dtype == part_ml.dtype == torch.float32 and part_o.numel() >= n * H * nsplit * rank
+                          and part_ml.numel() >= n * H * nsplit * 2), "latent_attention: partial results")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == H), "latent_attention: sink float32 [H]")
+    _check(lib().yalm_latent_attention(_p(q), _p(kv_step), _p(cache), _p(batch.token_seq), _p(batch.q_start),
+                                       _p(batch.seq_slot), _p(slot_pos), _p(out), _p(part_o), _p(part_ml),
+                                       dtype_code(q.dtype), n, H, rank, hd, capacity, int(window or 0), float(scale),
+                                       _p(sink), int(nsplit), 1 if mma else 0, pt, pps, npg, _stream()),
+           "latent_attention")
+
+
+def latent_prefill_usable(dtype: torch.dtype, dim: int, rd: int, vdim: int, rank: int, hd: int) -> bool:
+    return dtype in HALF_TYPES and bool(lib().yalm_latent_prefill_usable(dtype_code(dtype), dim, rd, vdim, rank, hd))
+
+
+def latent_prefill(q: torch.Tensor, kv: torch.Tensor, kv_step: torch.Tensor, batch, out: torch.Tensor, H: int,
+                   dim: int, rd: int, vdim: int, rank: int, hd: int, window: Optional[int], scale: float,
+                   sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_n: int = 1,
+                   gate_col0: int = 0, gate_mode: int = GATE_NONE) -> None:
+    """The expanded form, for sequences that start with this step: q [N, H, dim + rd] (rotated), kv
+    [N, H, dim + vdim] = (unrotated key | value) per head, kv_step [N, 2, 1, hd] with the shared rotated key
+    part at features rank .. rank + rd; out [N, H vdim], times sigmoid(gate)."""
+    n = batch.n_tokens
+    _need(q.dtype == kv.dtype == kv_step.dtype == out.dtype and q.is_contiguous() and kv.is_contiguous()
+          and kv_step.is_contiguous() and out.is_contiguous() and q.numel() == n * H * (dim + rd)
+          and kv.numel() == n * H * (dim + vdim) and kv_step.numel() == n * 2 * hd and out.numel() == n * H * vdim,
+          "latent_prefill: shapes")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == H), "latent_prefill: sink float32 [H]")
+    g = (None, 0, 0, 0, 0)
+    if gate is not None and gate_mode:
+        g = _columns(gate, gate_n, n, gate_col0, H if gate_mode == GATE_HEAD else H * vdim, "latent_prefill: gate slices")
+    _check(lib().yalm_latent_prefill(_p(q), _p(kv), _p(kv_step), _p(batch.q_start), _p(out), dtype_code(q.dtype),
+                                     batch.n_seqs, max(batch.q_lens), H, dim, rd, vdim, rank, hd, int(window or 0),
+                                     float(scale), _p(sink), g[0], int(gate_mode), *g[1:], _stream()), "latent_prefill")
+
+
+# ---- a state-space recurrence with one decay per head ------------------------------------------------
+def ssd_scan(act: torch.Tensor, dt: torch.Tensor, n_partials: int, col0: int, dt_bias: torch.Tensor,
+             a_log: torch.Tensor, d_skip: torch.Tensor, batch, state: torch.Tensor, out: torch.Tensor, H: int, G: int,
+             P: int, N: int) -> None:
+    """S_t = exp(-exp(a_log) dt_t) S_(t-1) + dt_t B_t x_t^T, out_t = S_t^T C_t + d_skip x_t per head (head h with
+    group h // (H / G)) over the step's tokens.  act float32 [N, H P + 2 G N] = (x | B | C); dt = softplus(column
+    col0 + h of the slices ``dt`` float32 [(s,) N, row] + dt_bias); ``state`` float32 [slots, H, P, N] is read at
+    the step's start and written at its end; out float32 [N, H P]."""
+    n = batch.n_tokens
+    _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, H * P + 2 * G * N)
+          and out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, H * P)
+          and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, P, N),
+          "ssd_scan: shapes")
+    for v in (dt_bias, a_log, d_skip):
+        _need(v.dtype == torch.float32 and v.numel() == H and v.is_contiguous(), "ssd_scan: float32 [H]")
+    src, s, stride, row, c = _columns(dt, n_partials, n, col0, H, "ssd_scan: step columns")
+    _check(lib().yalm_ssd_scan(_p(act), src, s, stride, row, c, _p(dt_bias), _p(a_log), _p(d_skip), _p(batch.q_start),
+                               _p(batch.seq_slot), _p(state), _p(out), n, batch.n_seqs, H, G, P, N, _stream()), "ssd_scan")
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, n_partials: int, col0: int, weight: torch.Tensor,
+                     out: torch.Tensor, groups: int, eps: float) -> None:
+    """out [N, inner] = y silu(z) with every one of ``groups`` equal parts of a row over its own root mean
+    square, times weight; y float32 [N, inner], z the ``inner`` columns from col0 of float32 slices [(s,) N, row]."""
+    n, inner = y.shape
+    _need(y.dtype == weight.dtype == torch.float32 and y.is_contiguous() and weight.numel() == inner
+          and out.is_contiguous() and tuple(out.shape) == (n, inner) and inner % groups == 0, "gated_group_norm: shapes")
+    _check(lib().yalm_gated_group_norm(_p(y), *_columns(z, n_partials, n, col0, inner, "gated_group_norm: gate columns"),
+                                       _p(weight), _p(out), dtype_code(out.dtype), n, inner, groups, float(eps),
+                                       _stream()), "gated_group_norm")
 
 
 GELU_TANH, TANH = 1, 2
@@ -1026,7 +1168,7 @@ def activation_rows(z: torch.Tensor, n_partials: int, out: torch.Tensor, act: in
 
 
 # ---- sublayer outputs normed before they join the residual stream -------------------------------------
-NORM_ABSENT, NORM_TANH, NORM_RMS, NORM_NONE = 0, 1, 2, 3
+NORM_ABSENT, NORM_TANH, NORM_RMS, NORM_NONE, NORM_LAYER = 0, 1, 2, 3, 4
 
 
 def norm_step(x: torch.Tensor, sets=(), post: Optional[tuple] = None, pre: Optional[tuple] = None,
@@ -1035,7 +1177,8 @@ def norm_step(x: torch.Tensor, sets=(), post: Optional[tuple] = None, pre: Optio
     """One pass over the rows of x float32 [N, dim]: x <- x + post(y), then h = pre(x).  y is the sum
     over ``sets`` (up to two (slices float32 [S, N, dim], S, factor)) of factor * sum of slices.  ``post``
     and ``pre`` are (kind, weight, bias, alpha, eps) with kind NORM_TANH (tanh(alpha v) w + b),
-    NORM_RMS (v / sqrt(mean v^2 + eps) w) or NORM_NONE, or None for a step without that half.  With
+    NORM_RMS (v / sqrt(mean v^2 + eps) w), NORM_LAYER ((v - mean) / sqrt(mean (v - mean)^2 + eps) w) or
+    NORM_NONE, or None for a step without that half.  With
     ``rows`` (int32 row numbers; no post half) only those rows are read: h [n_rows, dim]."""
     n, dim = x.shape
     _need(x.dtype == torch.float32 and x.is_contiguous(), "norm_step: x float32 [N, dim]")
@@ -1289,12 +1432,13 @@ def glu_clamp(gu: torch.Tensor, out: torch.Tensor, n_partials: int, alpha: float
 
 
 def routed_combine(x: torch.Tensor, y: torch.Tensor, pair_row: torch.Tensor, weight: torch.Tensor,
-                   top: int) -> None:
-    """x[t] += sum_j weight[t, j] * y[pair_row[t, j]]."""
+                   top: int, accumulate: bool = True) -> None:
+    """x[t] += (or, without ``accumulate``, =) sum_j weight[t, j] * y[pair_row[t, j]]."""
     n, dim = x.shape
     _need(x.dtype == y.dtype == weight.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous()
           and y.shape[1] == dim and pair_row.dtype == torch.int32, "routed_combine: shapes")
-    _check(lib().yalm_routed_combine(_p(x), _p(y), _p(pair_row), _p(weight), n, top, dim, _stream()),
+    _check(lib().yalm_routed_combine(_p(x), _p(y), _p(pair_row), _p(weight), n, top, dim,
+                                     1 if accumulate else 0, _stream()),
            "routed_combine")
 
 

@@ -15,7 +15,7 @@
 //                  output, as gemm_simt.cu).
 //   glu_clamp      y = g' sigmoid(alpha g') (u' + shift), g' = min(g, limit),
 //                  u' = clamp(u, -limit, limit); limit <= 0: no clamps.
-//   routed_combine x[t] += sum_j w[t, j] y[row(t, j)], in the order of j.
+//   routed_combine x[t] += (or =) sum_j w[t, j] y[row(t, j)], in the order of j.
 //
 // Nothing here depends on the order in which blocks run: a pair's row inside its expert's
 // group may differ from run to run, but every row is computed on its own and summed by
@@ -305,7 +305,7 @@ constexpr int RC_MAX_TOP = 256;
 
 __global__ void routed_combine_kernel(float* __restrict__ x, const float* __restrict__ y,
                                       const int* __restrict__ pair_row, const float* __restrict__ weight,
-                                      int top, int dim) {
+                                      int top, int dim, int accumulate) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -319,7 +319,7 @@ __global__ void routed_combine_kernel(float* __restrict__ x, const float* __rest
   // the rows of up to eight choices are loaded together, then added in the order of the choices
   if (dim % 4 == 0) {
     for (int i = threadIdx.x * 4; i < dim; i += blockDim.x * 4) {
-      float4 v = *reinterpret_cast<const float4*>(x + (size_t)t * dim + i);
+      float4 v = accumulate ? *reinterpret_cast<const float4*>(x + (size_t)t * dim + i) : make_float4(0.f, 0.f, 0.f, 0.f);
       for (int j0 = 0; j0 < top; j0 += 8) {
         float4 r[8];
 #pragma unroll
@@ -339,7 +339,7 @@ __global__ void routed_combine_kernel(float* __restrict__ x, const float* __rest
     return;
   }
   for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-    float v = x[(size_t)t * dim + i];
+    float v = accumulate ? x[(size_t)t * dim + i] : 0.f;
     for (int j0 = 0; j0 < top; j0 += 8) {
       float r[8];
 #pragma unroll
@@ -475,11 +475,11 @@ extern "C" int yalm_glu_clamp(const float* gu, int n_partials, long long partial
 }
 
 extern "C" int yalm_routed_combine(float* x, const float* y, const int* pair_row, const float* weight,
-                                   int n_tokens, int top, int dim, cudaStream_t stream) {
+                                   int n_tokens, int top, int dim, int accumulate, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (top <= 0 || top > RC_MAX_TOP) return -2;
   launch_pdl(routed_combine_kernel, dim3(n_tokens), dim3(dim >= 1024 ? 256 : 128), 0, stream, x, y,
-             pair_row, weight, top, dim);
+             pair_row, weight, top, dim, accumulate);
   YALM_LAUNCH_CHECK();
   return 0;
 }

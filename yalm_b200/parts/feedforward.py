@@ -122,6 +122,23 @@ class ClampedGLU:
         stream.add_linear(act, self.w_down)
 
 
+@register_feed_forward("clamped_glu")
+class ClampedGLUFeedForward(ClampedGLU):
+    """``ClampedGLU`` as a layer's dense feed-forward."""
+
+    def __init__(self, params: dict, rt):
+        super().__init__(params, rt, int(params["hidden_size"]))
+
+    def bind(self, tensors) -> None:
+        super().bind(tensors["gate"], tensors["up"], tensors["down"])
+
+    def flops(self, q_lens, past) -> float:
+        return super().flops(sum(q_lens))
+
+    def forward(self, h, batch, stream) -> None:
+        super().forward(h, stream, "ffn")
+
+
 @register_feed_forward("routed_experts")
 class RoutedExperts:
     """A mixture of experts: router logits z = Wr h and scores = softmax(z) over all experts
@@ -258,8 +275,7 @@ class RoutedExperts:
             if self.shared is not None:
                 raise RuntimeError("a shared expert beside a held stream is not supported")
             out = rt.buffer("routed_sum", (1, n, D), torch.float32)
-            out.zero_()
-            ops.routed_combine(out[0], y, pair_row, weight, top)
+            ops.routed_combine(out[0], y, pair_row, weight, top, accumulate=False)
             stream.pending, stream.n_pending = out, 1
             return
         ops.routed_combine(stream.resolve(), y, pair_row, weight, top)

@@ -47,6 +47,34 @@ class RMSNorm:
         return out
 
 
+@register_norm("layernorm")
+class LayerNorm:
+    """Layer norm with a weight and no bias: n(x) = (x - mean) / sqrt(var + eps) * w, var the mean of the
+    squared deviations, all in 32 bits.  As the norm of a sublayer's output it hands its ``form`` to
+    the stream."""
+
+    def __init__(self, params: dict, rt):
+        self.rt = rt
+        self.size = int(params["size"])
+        self.eps = float(params["eps"])
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensor_needs(self):
+        return {"weight": TensorNeed((self.size,), init="ones")}
+
+    def bind(self, tensors) -> None:
+        self.weight = self.rt.vector(tensors["weight"])
+
+    def form(self):
+        return (ops.NORM_LAYER, self.weight, None, 0.0, self.eps)
+
+    def __call__(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None,
+                 n_rows: Optional[int] = None, name: str = "normed") -> torch.Tensor:
+        n = stream.x.shape[0] if rows is None else int(n_rows)
+        out = self.rt.buffer(name, (n, self.size), self.rt.dtype)
+        return stream.read_norm(self.form(), out, rows=rows, n_rows=n_rows)
+
+
 @register_norm("dynamic_tanh")
 class DynamicTanh:
     """A norm that computes no mean and no variance: n(x) = tanh(alpha x) w + b, with a stored scalar
