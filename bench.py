@@ -481,7 +481,47 @@ SAMULORN_SIZES = {
                       head_dim=128, rot_dims=128, rec_width=4096, rec_blocks=16, ff=11008, experts=64, top=6,
                       groups=8, keep=4, expert_ff=1792, side_dim=256, pattern="dpd", vocab=32000),
 }
-DESIGNS = {"samulorn": (SAMULORN_SIZES, samulorn_config, samulorn_twin),
+def saralix_config(width, heads, dim, rot_dim, vdim, kv_rank, window, m_heads, m_vdim, state, groups, norm_groups, ff,
+                   experts, top, expert_ff, pattern, vocab):
+    """A Saralix configuration with layers of the sizes a served model has (random weights): ``pattern``
+    is a string of "l" (causal latent attention, experts), "s" (latent attention over a window with sinks, a
+    dense feed-forward) and "m" (mamba2, experts)."""
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+              "scale": float(dim + rot_dim) ** -0.5,
+              "rot": {"base": 1e4, "dims": rot_dim,
+                      "scaling": {"factor": 40.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}}
+    layer = {"l": {"type": "latent_attention", "mixer": latent, "mlp": moe},
+             "s": {"type": "latent_attention_2", "mixer": dict(latent, mask={"size": window}), "mlp": dense},
+             "m": {"type": "mamba2", "mlp": moe,
+                   "mixer": {"heads": m_heads, "vdim": m_vdim, "state": state, "groups": groups, "conv": 4,
+                             "norm_groups": norm_groups}}}
+    return {"architecture": "Saralix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": [layer[c] for c in pattern]}
+
+
+def saralix_twin(width, heads, dim, rot_dim, vdim, kv_rank, window, m_heads, m_vdim, state, groups, norm_groups, ff,
+                 experts, top, expert_ff, pattern, vocab):
+    """The closest model the library had before: the Llama / Mistral decoder with the same width,
+    layers and feed-forward and as many query heads of the value size over a quarter of the kv heads."""
+    return {"architectures": ["LlamaForCausalLM"], "hidden_size": width, "intermediate_size": ff,
+            "num_hidden_layers": len(pattern), "num_attention_heads": heads, "num_key_value_heads": heads // 4,
+            "head_dim": vdim, "vocab_size": vocab, "max_position_embeddings": 32768, "rms_norm_eps": 1e-6,
+            "rope_theta": 10000.0, "tie_word_embeddings": True, "hidden_act": "silu", "bos_token_id": 1,
+            "eos_token_id": 2}
+
+
+SARALIX_SIZES = {
+    "w2048-slml": dict(width=2048, heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=1024, m_heads=64,
+                       m_vdim=64, state=128, groups=8, norm_groups=8, ff=5632, experts=32, top=4, expert_ff=1408,
+                       pattern="slml", vocab=32000),
+    "w4096-slm": dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048, m_heads=128,
+                      m_vdim=64, state=128, groups=8, norm_groups=8, ff=11008, experts=64, top=6, expert_ff=1792,
+                      pattern="slm", vocab=32000),
+}
+DESIGNS = {"saralix": (SARALIX_SIZES, saralix_config, saralix_twin),
+           "samulorn": (SAMULORN_SIZES, samulorn_config, samulorn_twin),
            "golulix": (DESIGN_SIZES, golulix_config, dense_twin),
            "rudazen": (RUDAZEN_SIZES, rudazen_config, rudazen_twin),
            "nekotar": (NEKOTAR_SIZES, nekotar_config, nekotar_twin)}
@@ -631,7 +671,7 @@ def main():
                          "beside the dense decoder at equal sizes (random weights, a few layers)")
     ap.add_argument("--design", default="golulix", choices=sorted(DESIGNS),
                     help="with --compare-designs: which design runs beside the dense decoder")
-    ap.add_argument("--design-size", default=None, choices=sorted(set(DESIGN_SIZES) | set(RUDAZEN_SIZES) | set(NEKOTAR_SIZES) | set(SAMULORN_SIZES)),
+    ap.add_argument("--design-size", default=None, choices=sorted(set(DESIGN_SIZES) | set(RUDAZEN_SIZES) | set(NEKOTAR_SIZES) | set(SAMULORN_SIZES) | set(SARALIX_SIZES)),
                     help="with --compare-designs: one of the design's sizes instead of all")
     args = ap.parse_args()
 

@@ -354,8 +354,9 @@ int yalm_latent_attention_mma_usable(int dtype, int rank, int hd);
 int yalm_latent_attention(const void* q, const void* kv_step, const void* cache, const int* token_seq,
                           const int* q_start, const int* seq_slot, const int* slot_pos, void* out,
                           float* part_o, float* part_ml, int dtype, int n_tokens, int H, int rank, int hd,
-                          int capacity, int window, float scale, const float* sink, int nsplit, int mma,
-                          const int* page_table, int pages_per_slot, int n_pages, cudaStream_t stream);
+                          int capacity, int window, float scale, const float* sink, int nsplit, int per_split,
+                          int mma, const int* page_table, int pages_per_slot, int n_pages,
+                          cudaStream_t stream);
 int yalm_latent_prefill_usable(int dtype, int dim, int rd, int vdim, int rank, int hd);
 int yalm_latent_prefill(const void* q, const void* kv, const void* kv_step, const int* q_start, void* out,
                         int dtype, int n_seqs, int max_q_len, int H, int dim, int rd, int vdim, int rank,

@@ -4,10 +4,11 @@
 //
 //  * attn_latent_mma (16-bit): the absorbed form, a decode step's or a portion's queries over the
 //    cached rows.  A block takes 16 heads of one token over one run of its keys; the rows -- keys
-//    and values at once -- come in tiles of 64 through two cp.async buffers.  S = q K^T by
-//    mma.sync (the 16 heads are the rows of a tile, a warp takes 8 keys), softmax by 16 threads per
-//    head, O += P C with every weight as three 16-bit terms (all its bits), a warp per part of the
-//    columns.  A row is read from memory once for all heads of the group.
+//    and values at once -- come in tiles of 32 through two cp.async buffers, small enough for two
+//    blocks to share an SM: one's softmax and barriers run under the other's products.  S = q K^T by
+//    mma.sync (the 16 heads are the rows of a tile; a warp takes 8 keys and half of the features),
+//    softmax by 16 threads per head, O += P C with every weight as three 16-bit terms (all its bits), a
+//    warp per part of the columns.  A row is read from memory once for all heads of the group.
 //  * attn_latent_fma: the same with 32-bit FMA on any storage type: the 32-bit path, and row sizes
 //    that the kernel above does not take.
 //  * attn_latent_prefill (16-bit): the expanded form for whole prompts: per head keys
@@ -65,7 +66,7 @@ struct LatentRows {
   const void *kv_step, *cache;
   const int *token_seq, *q_start, *seq_slot, *slot_pos;
   const int* page_table;
-  int pps, n_pages, capacity, hd, rank, H, window, nsplit;
+  int pps, n_pages, capacity, hd, rank, H, window, nsplit, per;      // per: keys of a split
   float scale_log2;
   const float* sink;         // [H] or null
 };
@@ -74,12 +75,10 @@ struct LatentOut {
   float *part_o, *part_ml;   // else [tokens][H][nsplit][rank] and [tokens][H][nsplit][2] (maximum in log2 units, sum)
 };
 
-// the run of keys of one split: whole tiles of 64
-__device__ __forceinline__ void split_range(int lo, int pos, int nsplit, int split, int& k0, int& k1) {
-  const int tiles = (pos - lo + 64) / 64;
-  const int per = (tiles + nsplit - 1) / nsplit * 64;
-  k0 = lo + split * per;
-  k1 = min(k0 + per, pos + 1);
+// the run of keys of one split; the last split takes whatever is left
+__device__ __forceinline__ void split_range(const LatentRows& a, int lo, int pos, int split, int& k0, int& k1) {
+  k0 = lo + split * a.per;
+  k1 = split == a.nsplit - 1 ? pos + 1 : min(k0 + a.per, pos + 1);
 }
 template <typename T>
 __device__ __forceinline__ const T* latent_row(const LatentRows& a, int key, int past, int qs, int slot) {
@@ -88,21 +87,21 @@ __device__ __forceinline__ const T* latent_row(const LatentRows& a, int key, int
          kv_row_offset(a.page_table, a.pps, a.n_pages, slot, 0, 1, a.capacity, key % a.capacity, a.hd);
 }
 
-constexpr int LA_HEADS = 16, LA_KEYS = 64, LA_WARPS = 8;
+constexpr int LA_HEADS = 16, LA_KEYS = 32, LA_WARPS = 8;
 constexpr int LA_SP = LA_KEYS + 4;                     // pitch of the scores (floats)
 constexpr int LA_PP = LA_KEYS + 8;                     // pitch of the weights (16-bit)
 
 // NT: 8-column tiles per warp; rank <= 64 NT.  grid (splits, head groups, tokens)
 template <typename T, int NT>
-__global__ void __launch_bounds__(LA_WARPS * 32)
+__global__ void __launch_bounds__(LA_WARPS * 32, 2)
 attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t la_smem[];
   const int hd = a.hd, lds = hd + 8;
   T* qs_ = reinterpret_cast<T*>(la_smem);              // [16][lds]
-  T* rows = qs_ + LA_HEADS * lds;                      // two tiles [64][lds]
+  T* rows = qs_ + LA_HEADS * lds;                      // two tiles [32][lds]
   T* ps = rows + 2 * LA_KEYS * lds + 32;               // weights, three terms [3][16][LA_PP]
-  float* ss = reinterpret_cast<float*>(ps + 3 * LA_HEADS * LA_PP);        // scores [16][LA_SP]
+  float* ss = reinterpret_cast<float*>(ps + 3 * LA_HEADS * LA_PP);        // scores of either half [2][16][LA_SP]
   __shared__ float corr_s[LA_HEADS], l_s[LA_HEADS];
   const int t = blockIdx.z, h0 = blockIdx.y * LA_HEADS, split = blockIdx.x;
   const int nh = min(LA_HEADS, a.H - h0);
@@ -111,7 +110,7 @@ attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
   const int past = a.slot_pos[slot], pos = past + (t - qs);
   const int lo = first_visible(pos, a.window);
   int k0, k1;
-  split_range(lo, pos, a.nsplit, split, k0, k1);
+  split_range(a, lo, pos, split, k0, k1);
   pdl_wait();
   if (k0 >= k1 && a.nsplit > 1) {                      // a split without keys (the first always has one)
     if (threadIdx.x < nh) {
@@ -122,24 +121,24 @@ attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
     return;
   }
   const int pieces = hd / 8;
+  auto issue = [&](int base, int buf) {
+    const int r = threadIdx.x >> 3, key = base + r;
+    const bool on = key < k1;
+    const T* src = on ? latent_row<T>(a, key, past, qs, slot) : q;
+    T* dst = rows + (size_t)buf * LA_KEYS * lds + r * lds;
+    for (int c = threadIdx.x & 7; c < pieces; c += 8) cp16(dst + c * 8, src + (on ? c * 8 : 0), on ? 16 : 0);
+    cp_commit();
+  };
   for (int i = threadIdx.x; i < LA_HEADS * pieces; i += blockDim.x) {
     const int r = i / pieces, c = i - r * pieces;
     const bool on = r < nh;
     cp16(qs_ + r * lds + c * 8, q + ((size_t)t * a.H + h0 + (on ? r : 0)) * hd + c * 8, on ? 16 : 0);
   }
-  auto issue = [&](int base, int buf) {
-    const int r = threadIdx.x >> 2, key = base + r;
-    const bool on = key < k1;
-    const T* src = on ? latent_row<T>(a, key, past, qs, slot) : q;
-    T* dst = rows + (size_t)buf * LA_KEYS * lds + r * lds;
-    for (int c = threadIdx.x & 3; c < pieces; c += 4) cp16(dst + c * 8, src + (on ? c * 8 : 0), on ? 16 : 0);
-    cp_commit();
-  };
   issue(k0, 0);
   float o[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  // softmax: 16 threads per head, four keys each
+  // softmax: 16 threads per head, two keys each
   const int sh = threadIdx.x >> 4, sk = threadIdx.x & 15;
   float m = -INFINITY, l = 0.f;
   if (a.sink != nullptr && split == 0 && sh < nh) {
@@ -148,19 +147,22 @@ attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
   }
   const int g = lane >> 2, t4 = lane & 3;
   const int n_tiles = (k1 - k0 + LA_KEYS - 1) / LA_KEYS;
+  const int nk = hd / 16, nk_half = ((nk + 3) / 4) * 2;            // the first half has an even number of steps
+  const int kh = warp >> 2, kt = warp & 3;             // this warp's half of the features and its 8 keys
+  const int kk0 = kh ? nk_half : 0, kk1 = kh ? nk : min(nk_half, nk);
   for (int it = 0; it < n_tiles; ++it) {
     const int base = k0 + it * LA_KEYS;
     cp_wait<0>();
     __syncthreads();                                   // the tile has landed; the other buffer is no longer read
     if (it + 1 < n_tiles) issue(base + LA_KEYS, (it + 1) & 1);
     const T* tile = rows + (size_t)(it & 1) * LA_KEYS * lds;
-    {                                                  // S: this warp's 8 keys, 16 heads
+    {
       float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
       const uint32_t qa = smem_u32(qs_ + (lane & 15) * lds + (lane >> 4) * 8);
-      const uint32_t kb = smem_u32(tile + (warp * 8 + (lane & 7)) * lds + (lane >> 3) * 8);
-      const int nk = hd / 16;
-      int kk = 0;
-      for (; kk + 2 <= nk; kk += 2) {
+      const uint32_t kb = smem_u32(tile + (kt * 8 + (lane & 7)) * lds + (lane >> 3) * 8);
+      int kk = kk0;
+#pragma unroll 4
+      for (; kk + 2 <= kk1; kk += 2) {
         uint32_t qf[4], qg[4], kf[4];
         ldsm_x4(kf, kb + kk * 32);
         ldsm_x4(qf, qa + kk * 32);
@@ -168,66 +170,67 @@ attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
         mma16<T>(s0, qf, kf[0], kf[1]);
         mma16<T>(s1, qg, kf[2], kf[3]);
       }
-      if (kk < nk) {
+      if (kk < kk1) {
         uint32_t qf[4], kf[4];
         ldsm_x4(kf, kb + kk * 32);                     // the upper half lies in the pad and is not used
         ldsm_x4(qf, qa + kk * 32);
         mma16<T>(s0, qf, kf[0], kf[1]);
       }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = warp * 8 + 2 * t4 + (e & 1);
-        const float v = (s0[e] + s1[e]) * a.scale_log2;
-        ss[(g + 8 * (e >> 1)) * LA_SP + key] = base + key < k1 ? v : -INFINITY;
-      }
+      float* sd = ss + kh * LA_HEADS * LA_SP + kt * 8 + 2 * t4;
+      *reinterpret_cast<float2*>(sd + g * LA_SP) = make_float2(s0[0] + s1[0], s0[1] + s1[1]);
+      *reinterpret_cast<float2*>(sd + (g + 8) * LA_SP) = make_float2(s0[2] + s1[2], s0[3] + s1[3]);
     }
     __syncthreads();
     {
-      const float4 v = *reinterpret_cast<const float4*>(ss + sh * LA_SP + sk * 4);
-      float mx = fmaxf(fmaxf(v.x, v.y), fmaxf(v.z, v.w));
+      const float2 u = *reinterpret_cast<const float2*>(ss + sh * LA_SP + sk * 2);
+      const float2 w = *reinterpret_cast<const float2*>(ss + (LA_HEADS + sh) * LA_SP + sk * 2);
+      const int key = base + sk * 2;
+      const float x0 = key < k1 ? (u.x + w.x) * a.scale_log2 : -INFINITY;
+      const float x1 = key + 1 < k1 ? (u.y + w.y) * a.scale_log2 : -INFINITY;
+      float mx = fmaxf(x0, x1);
 #pragma unroll
       for (int off = 8; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
       const float mn = fmaxf(m, mx);                   // a tile has at least one key
       const float corr = exp2f(m - mn);                // exp2(-inf) = 0 on the first
       m = mn;
-      const float p0 = exp2f(v.x - mn), p1 = exp2f(v.y - mn), p2 = exp2f(v.z - mn), p3 = exp2f(v.w - mn);
-      l = l * corr + ((p0 + p1) + (p2 + p3));
+      const float p0 = exp2f(x0 - mn), p1 = exp2f(x1 - mn);
+      l = l * corr + (p0 + p1);
       if (sk == 0) corr_s[sh] = corr;
-      uint2 hi, mid, low;
-      three_terms<T>(p0, p1, hi.x, mid.x, low.x);
-      three_terms<T>(p2, p3, hi.y, mid.y, low.y);
-      T* p = ps + sh * LA_PP + sk * 4;
-      *reinterpret_cast<uint2*>(p) = hi;
-      *reinterpret_cast<uint2*>(p + LA_HEADS * LA_PP) = mid;
-      *reinterpret_cast<uint2*>(p + 2 * LA_HEADS * LA_PP) = low;
+      uint32_t hi, mid, low;
+      three_terms<T>(p0, p1, hi, mid, low);
+      uint32_t* p = reinterpret_cast<uint32_t*>(ps + sh * LA_PP + sk * 2);
+      p[0] = hi;
+      p[LA_HEADS * LA_PP / 2] = mid;
+      p[LA_HEADS * LA_PP] = low;
     }
     __syncthreads();
     {
       const float c0 = corr_s[g], c1 = corr_s[g + 8];
+      if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-      for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+        for (int i = 0; i < NT; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+      }
       const uint32_t pa = smem_u32(ps + (lane & 15) * LA_PP + (lane >> 4) * 8);
       const uint32_t va = smem_u32(tile + ((lane >> 3 & 1) * 8 + (lane & 7)) * lds + (lane >> 4) * 8);
 #pragma unroll
       for (int kk = 0; kk < LA_KEYS / 16; ++kk) {
-        uint32_t hi[4], mid[4], low[4];
-        ldsm_x4(hi, pa + kk * 32);
-        ldsm_x4(mid, pa + kk * 32 + LA_HEADS * LA_PP * 2);
-        ldsm_x4(low, pa + kk * 32 + 2 * LA_HEADS * LA_PP * 2);
+        uint32_t p[3][4], r[NT / 2][4];                // the small terms first
+        ldsm_x4(p[2], pa + kk * 32);
+        ldsm_x4(p[1], pa + kk * 32 + LA_HEADS * LA_PP * 2);
+        ldsm_x4(p[0], pa + kk * 32 + 2 * LA_HEADS * LA_PP * 2);
 #pragma unroll
         for (int n2 = 0; n2 < NT / 2; ++n2) {
-          const int col = warp * NT * 8 + n2 * 16;
-          if (col < a.rank) {                          // rank <= hd and hd is a multiple of 16: in bounds
-            uint32_t r[4];
-            ldsm_x4_trans(r, va + (uint32_t)(kk * 16 * lds + col) * 2);
-            mma16<T>(o[2 * n2], low, r[0], r[1]);
-            mma16<T>(o[2 * n2 + 1], low, r[2], r[3]);
-            mma16<T>(o[2 * n2], mid, r[0], r[1]);
-            mma16<T>(o[2 * n2 + 1], mid, r[2], r[3]);
-            mma16<T>(o[2 * n2], hi, r[0], r[1]);
-            mma16<T>(o[2 * n2 + 1], hi, r[2], r[3]);
-          }
+          const int col = warp * NT * 8 + n2 * 16;     // rank <= hd and hd is a multiple of 16: in bounds
+          if (col < a.rank) ldsm_x4_trans(r[n2], va + (uint32_t)(kk * 16 * lds + col) * 2);
         }
+#pragma unroll
+        for (int term = 0; term < 3; ++term)
+#pragma unroll
+          for (int n2 = 0; n2 < NT / 2; ++n2)
+            if (warp * NT * 8 + n2 * 16 < a.rank) {
+              mma16<T>(o[2 * n2], p[term], r[n2][0], r[n2][1]);
+              mma16<T>(o[2 * n2 + 1], p[term], r[n2][2], r[n2][3]);
+            }
       }
     }
   }
@@ -254,8 +257,12 @@ attn_latent_mma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
       const float x = o[i][2 * half], y = o[i][2 * half + 1];
       if (a.nsplit > 1) {
         float* dst = o_.part_o + (((size_t)t * a.H + h0 + head) * a.nsplit + split) * a.rank + col;
-        dst[0] = x;
-        if (col + 1 < a.rank) dst[1] = y;
+        if ((a.rank & 1) == 0) {
+          *reinterpret_cast<float2*>(dst) = make_float2(x, y);
+        } else {
+          dst[0] = x;
+          if (col + 1 < a.rank) dst[1] = y;
+        }
       } else {                                         // hd is a multiple of 16: col + 1 < hd
         *reinterpret_cast<uint32_t*>(reinterpret_cast<T*>(o_.out) + ((size_t)t * a.H + h0 + head) * hd + col) =
             pack2<T>(x * inv, y * inv);
@@ -281,7 +288,7 @@ attn_latent_fma_kernel(const T* __restrict__ q, LatentRows a, LatentOut o_) {
   const int past = a.slot_pos[slot], pos = past + (t - qs);
   const int lo = first_visible(pos, a.window);
   int k0, k1;
-  split_range(lo, pos, a.nsplit, split, k0, k1);
+  split_range(a, lo, pos, split, k0, k1);
   pdl_wait();
   if (k0 >= k1 && a.nsplit > 1) {
     if (threadIdx.x < nh) {
@@ -505,8 +512,10 @@ attn_latent_prefill_kernel(PromptArgs a) {
       const float corr = exp2f(m[rr] - sub);
       m[rr] = mn;
       l[rr] *= corr;
+      if (__any_sync(0xffffffffu, corr != 1.f)) {        // most blocks raise no maximum
 #pragma unroll
-      for (int i = 0; i < 2 * NV; ++i) { o[i][2 * rr] *= corr; o[i][2 * rr + 1] *= corr; }
+        for (int i = 0; i < 2 * NV; ++i) { o[i][2 * rr] *= corr; o[i][2 * rr + 1] *= corr; }
+      }
       float sum = 0.f;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt)
@@ -580,7 +589,7 @@ using namespace yalm;
   } while (0)
 
 static size_t latent_mma_smem(int hd) {
-  return ((size_t)(LA_HEADS + 2 * LA_KEYS) * (hd + 8) + 32 + 3 * LA_HEADS * LA_PP) * 2 + (size_t)LA_HEADS * LA_SP * 4;
+  return ((size_t)(LA_HEADS + 2 * LA_KEYS) * (hd + 8) + 32 + 3 * LA_HEADS * LA_PP) * 2 + (size_t)2 * LA_HEADS * LA_SP * 4;
 }
 
 // whether yalm_latent_attention runs on tensor cores for these sizes
@@ -591,19 +600,19 @@ extern "C" int yalm_latent_attention_mma_usable(int dtype, int rank, int hd) {
 
 // The absorbed form.  q, out [tokens][H][hd]; kv_step [tokens][2][hd]; cache [slots][1][capacity][hd] or
 // pages; with nsplit > 1 part_o [tokens][H][nsplit][rank] and part_ml [tokens][H][nsplit][2] instead of
-// out.  sink [H] float32 or null.  mma: 0 runs the FMA kernel whatever the type.
+// out, split s the keys from per_split s on (those of a query that sees fewer keys stay empty).  sink [H] float32 or null.  mma: 0 runs the FMA kernel whatever the type.
 extern "C" int yalm_latent_attention(const void* q, const void* kv_step, const void* cache, const int* token_seq,
                                      const int* q_start, const int* seq_slot, const int* slot_pos, void* out,
                                      float* part_o, float* part_ml, int dtype, int n_tokens, int H, int rank,
                                      int hd, int capacity, int window, float scale, const float* sink, int nsplit,
-                                     int mma, const int* page_table, int pages_per_slot, int n_pages,
+                                     int per_split, int mma, const int* page_table, int pages_per_slot, int n_pages,
                                      cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (H <= 0 || rank <= 0 || rank > 256 * LF_MAX_COLS || hd < rank || hd > 2048 || capacity <= 0 || window < 0) return -2;
-  if (nsplit < 1 || nsplit > 64 || !(scale > 0.f)) return -5;
+  if (nsplit < 1 || nsplit > 64 || per_split < 0 || (nsplit > 1 && per_split <= 0) || !(scale > 0.f)) return -5;
   if (n_tokens > 65535 || (H + LF_HEADS - 1) / LF_HEADS > 65535) return -4;
   const LatentRows a = {kv_step, cache, token_seq, q_start, seq_slot, slot_pos, page_table, pages_per_slot, n_pages,
-                        capacity, hd, rank, H, window, nsplit, scale * LOG2E, sink};
+                        capacity, hd, rank, H, window, nsplit, per_split, scale * LOG2E, sink};
   const LatentOut o = {out, part_o, part_ml};
   if (mma && yalm_latent_attention_mma_usable(dtype, rank, hd)) {
     const dim3 grid(nsplit, (H + LA_HEADS - 1) / LA_HEADS, n_tokens);

@@ -174,6 +174,116 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
   }
 }
 
+// The same step with the row in registers: a thread owns E groups of four neighbouring features (every
+// blockDim.x-th group), so that nothing but the sums goes through shared memory.  One barrier per sum:
+// every sum has partial results of its own, which each warp adds up for itself.
+__device__ __forceinline__ float row_sum(float v, float* part) {
+  const int lane = threadIdx.x & 31;
+  v = warp_sum(v);
+  if (lane == 0) part[threadIdx.x >> 5] = v;
+  __syncthreads();
+  return warp_sum(lane < (int)(blockDim.x >> 5) ? part[lane] : 0.f);
+}
+
+template <typename T, int E>
+__global__ void norm_step_reg_kernel(float* __restrict__ x, SliceSet A, SliceSet B, NormForm post, NormForm pre,
+                                     T* __restrict__ h, const int* __restrict__ rows, int dim) {
+  pdl_launch_dependents();
+  __shared__ float parts[4][32];
+  pdl_wait();
+  const size_t t = rows != nullptr ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x;
+  float* xr = x + t * dim;
+  const int nv = dim >> 2;
+  float v[E][4], y[E][4];
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = threadIdx.x + e * blockDim.x;
+    const float4 a = i < nv ? reinterpret_cast<const float4*>(xr)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    v[e][0] = a.x; v[e][1] = a.y; v[e][2] = a.z; v[e][3] = a.w;
+  }
+  if (post.kind) {
+    float s1 = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = (threadIdx.x + e * blockDim.x) * 4;
+      float4 ya = make_float4(0.f, 0.f, 0.f, 0.f), yb = ya;
+      if (i < dim) {
+        if (A.p != nullptr) ya = slices4(A.p + t * dim + i, A.n, A.stride);
+        if (B.p != nullptr) yb = slices4(B.p + t * dim + i, B.n, B.stride);
+      }
+      y[e][0] = fmaf(B.factor, yb.x, A.factor * ya.x); y[e][1] = fmaf(B.factor, yb.y, A.factor * ya.y);
+      y[e][2] = fmaf(B.factor, yb.z, A.factor * ya.z); y[e][3] = fmaf(B.factor, yb.w, A.factor * ya.w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s1 += post.kind == 4 ? y[e][j] : y[e][j] * y[e][j];
+    }
+    float r = 1.f, mean = 0.f;
+    if (post.kind == 2) r = 1.0f / sqrtf(row_sum(s1, parts[0]) / (float)dim + post.eps);
+    if (post.kind == 4) {
+      mean = row_sum(s1, parts[0]) / (float)dim;
+      float s2 = 0.f;
+#pragma unroll
+      for (int e = 0; e < E; ++e)
+        if (threadIdx.x + e * blockDim.x < nv)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) { const float d = y[e][j] - mean; s2 += d * d; }
+      r = 1.0f / sqrtf(row_sum(s2, parts[1]) / (float)dim + post.eps);
+    }
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      const int i = threadIdx.x + e * blockDim.x;
+      if (i < nv) {
+        if (post.kind == 1) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[e][j] += apply_tanh_form(post, y[e][j], 4 * i + j);
+        } else if (post.kind == 3) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[e][j] += y[e][j];
+        } else {                                           // mean is zero in the rms form
+          const float4 w = reinterpret_cast<const float4*>(post.w)[i];
+          v[e][0] += (y[e][0] - mean) * r * w.x; v[e][1] += (y[e][1] - mean) * r * w.y;
+          v[e][2] += (y[e][2] - mean) * r * w.z; v[e][3] += (y[e][3] - mean) * r * w.w;
+        }
+        reinterpret_cast<float4*>(xr)[i] = make_float4(v[e][0], v[e][1], v[e][2], v[e][3]);
+      }
+    }
+  }
+  if (!pre.kind) return;
+  float r = 1.f, mean = 0.f;
+  if (pre.kind == 2 || pre.kind == 4) {
+    if (pre.kind == 4) {
+      float s1 = 0.f;
+#pragma unroll
+      for (int e = 0; e < E; ++e)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s1 += v[e][j];         // groups beyond the row hold zeros
+      mean = row_sum(s1, parts[2]) / (float)dim;
+    }
+    float s2 = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e)
+      if (threadIdx.x + e * blockDim.x < nv)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { const float d = v[e][j] - mean; s2 += d * d; }
+    r = 1.0f / sqrtf(row_sum(s2, parts[3]) / (float)dim + pre.eps);
+  }
+  T* out = h + (size_t)blockIdx.x * dim;
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = threadIdx.x + e * blockDim.x;
+    if (i >= nv) continue;
+    float o[4];
+    if (pre.kind == 2 || pre.kind == 4) {
+      const float4 w = reinterpret_cast<const float4*>(pre.w)[i];
+      o[0] = (v[e][0] - mean) * r * w.x; o[1] = (v[e][1] - mean) * r * w.y;
+      o[2] = (v[e][2] - mean) * r * w.z; o[3] = (v[e][3] - mean) * r * w.w;
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[j] = pre.kind == 1 ? apply_tanh_form(pre, v[e][j], 4 * i + j) : v[e][j];
+    }
+    store4<T>(out + 4 * i, o[0], o[1], o[2], o[3]);
+  }
+}
+
 constexpr int CONV_MAX_TAPS = 8;
 
 struct ConvArgs {
@@ -263,6 +373,75 @@ __global__ void short_conv_kernel(ConvArgs a, const int* __restrict__ token_seq,
   }
 }
 
+// The same for many tokens of a product in one slice: a thread owns four neighbouring channels
+// (16-byte accesses; channels, pitches and columns in multiples of four), 32-bit output only.
+__device__ __forceinline__ float4 conv_input4(const ConvArgs& a, int token, int c) {
+  float4 v = *reinterpret_cast<const float4*>(a.src + (size_t)token * a.src_row + a.src_col0 + c);
+  if (a.in_bias != nullptr) {
+    const float4 b = *reinterpret_cast<const float4*>(a.in_bias + c);
+    v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+  }
+  return v;
+}
+__device__ __forceinline__ void fma4(float4& y, const float* w, int stride, const float4& u) {
+  y.x = fmaf(w[0], u.x, y.x); y.y = fmaf(w[stride], u.y, y.y);
+  y.z = fmaf(w[2 * stride], u.z, y.z); y.w = fmaf(w[3 * stride], u.w, y.w);
+}
+template <int TAPS, int RUN>
+__global__ void __launch_bounds__(128)
+short_conv4_kernel(ConvArgs a, const int* __restrict__ token_seq, const int* __restrict__ q_start,
+                   const int* __restrict__ seq_slot, float* __restrict__ out32, int out_row, int out_col0,
+                   int n_tokens) {
+  pdl_launch_dependents();
+  const int t_first = blockIdx.x * RUN;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (c >= a.channels) return;
+  float w[4 * TAPS];                                     // [channel][tap]
+#pragma unroll
+  for (int k = 0; k < 4 * TAPS; ++k) w[k] = a.w[(size_t)c * TAPS + k];
+  float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (a.out_bias != nullptr) bias = make_float4(a.out_bias[c], a.out_bias[c + 1], a.out_bias[c + 2], a.out_bias[c + 3]);
+  pdl_wait();
+  float4 cur[RUN];
+#pragma unroll
+  for (int j = 0; j < RUN; ++j) cur[j] = conv_input4(a, min(t_first + j, n_tokens - 1), c);
+  constexpr int before = TAPS - 1;
+  float4 win[before];
+#pragma unroll
+  for (int j = 0; j < RUN; ++j) {
+    const int t = t_first + j;
+    if (t < n_tokens) {
+      const int b = token_seq[t];
+      const int qs = q_start[b], local = t - qs;
+      float* st = a.state + (size_t)seq_slot[b] * before * a.channels + c;
+      if (j == 0 || local == 0) {
+#pragma unroll
+        for (int k = 0; k < before; ++k) {
+          const int idx = local - before + k;
+          win[k] = idx >= 0 ? conv_input4(a, qs + idx, c)
+                            : *reinterpret_cast<const float4*>(st + (size_t)(before + idx) * a.channels);
+        }
+      }
+      float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < before; ++k) fma4(y, w + k, TAPS, win[k]);
+      fma4(y, w + before, TAPS, cur[j]);
+      y.x += bias.x; y.y += bias.y; y.z += bias.z; y.w += bias.w;
+      if (a.silu) {
+        y.x /= 1.0f + expf(-y.x); y.y /= 1.0f + expf(-y.y); y.z /= 1.0f + expf(-y.z); y.w /= 1.0f + expf(-y.w);
+      }
+      *reinterpret_cast<float4*>(out32 + (size_t)t * out_row + out_col0 + c) = y;
+#pragma unroll
+      for (int k = 0; k + 1 < before; ++k) win[k] = win[k + 1];
+      win[before - 1] = cur[j];
+      if (q_start[b + 1] - qs == 1) {                    // a sequence that brings one token: the state moves on here
+#pragma unroll
+        for (int k = 0; k < before; ++k) *reinterpret_cast<float4*>(st + (size_t)k * a.channels) = win[k];
+      }
+    }
+  }
+}
+
 // grid (sequences, parts of the channels): the step's last taps - 1 inputs of every sequence that
 // brought more than one token (some of them the state's own, when it brought fewer than taps - 1)
 __global__ void short_conv_state_kernel(ConvArgs a, const int* __restrict__ q_start,
@@ -322,10 +501,30 @@ extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, fl
   const NormForm pre = {pre_kind, pre_w, pre_b, pre_alpha, pre_eps};
   const bool vec = dim % 4 == 0 && (sa & 3) == 0 && (sb & 3) == 0 &&
                    ((((uintptr_t)x) | ((uintptr_t)a) | ((uintptr_t)b) | ((uintptr_t)h)) & 15) == 0;
+  const dim3 grid(n_rows);
+  if (vec && dim <= 8192 && ((((uintptr_t)post_w) | ((uintptr_t)pre_w)) & 15) == 0) {
+    // many rows: four groups of four features per thread, so that many rows are in flight on an SM; few: one
+    const int groups = dim / 4;
+    const int e = n_rows >= 512 && groups >= 256 ? 4 : groups > 1024 ? 2 : 1;
+    const dim3 block(((groups + e - 1) / e + 31) / 32 * 32);
+#define YALM_NSR(T)                                                                                            \
+  do {                                                                                                         \
+    if (e == 4) launch_pdl(norm_step_reg_kernel<T, 4>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim); \
+    else if (e == 2) launch_pdl(norm_step_reg_kernel<T, 2>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim); \
+    else launch_pdl(norm_step_reg_kernel<T, 1>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim);  \
+  } while (0)
+    if (h_dtype == DT_F32) YALM_NSR(float);
+    else if (h_dtype == DT_BF16) YALM_NSR(__nv_bfloat16);
+    else if (h_dtype == DT_F16) YALM_NSR(__half);
+    else return -3;
+#undef YALM_NSR
+    YALM_LAUNCH_CHECK();
+    return 0;
+  }
   int threads = ((vec ? dim / 4 : dim) + 31) / 32 * 32;
   if (threads > 512) threads = 512;
   if (n_rows <= 64 && dim >= 8192 && !vec) threads = 1024;
-  const dim3 grid(n_rows), block(threads);
+  const dim3 block(threads);
   const size_t smem = (size_t)dim * sizeof(float);
 #define YALM_NS1(T, V)                                                                                 \
   do {                                                                                                \
@@ -376,6 +575,9 @@ extern "C" int yalm_short_conv(const float* src, int n_partials, long long parti
   const int run = n_tokens >= 1024 ? 8 : 1;
   const dim3 grid((n_tokens + run - 1) / run, parts), block(threads);
   const int b16 = out16 != nullptr ? block16 : channels;
+  const bool four = run == 8 && n_partials == 1 && out16 == nullptr && channels % 4 == 0 && src_row % 4 == 0 &&
+                    src_col0 % 4 == 0 && out_row % 4 == 0 && out_col0 % 4 == 0 &&
+                    ((((uintptr_t)src) | ((uintptr_t)in_bias) | ((uintptr_t)state) | ((uintptr_t)out32)) & 15) == 0;
 #define YALM_CONV(T, TAPS)                                                                                \
   do {                                                                                                    \
     if (run == 8 && n_partials == 1)                                                                      \
@@ -400,7 +602,23 @@ extern "C" int yalm_short_conv(const float* src, int n_partials, long long parti
       default: YALM_CONV(T, 8); break;                                                                  \
     }                                                                                                   \
   } while (0)
-  if (out16 == nullptr || out16_dtype == DT_F32) YALM_CONV_T(float);
+  if (four) {
+    const dim3 grid4((n_tokens + 7) / 8, (channels / 4 + 127) / 128), block4(128);
+#define YALM_CONV4(TAPS)                                                                                   \
+  launch_pdl(short_conv4_kernel<TAPS, 8>, grid4, block4, 0, stream, a, token_seq, q_start, seq_slot, out32, \
+             out_row, out_col0, n_tokens)
+    switch (taps) {
+      case 2: YALM_CONV4(2); break;
+      case 3: YALM_CONV4(3); break;
+      case 4: YALM_CONV4(4); break;
+      case 5: YALM_CONV4(5); break;
+      case 6: YALM_CONV4(6); break;
+      case 7: YALM_CONV4(7); break;
+      default: YALM_CONV4(8); break;
+    }
+#undef YALM_CONV4
+  }
+  else if (out16 == nullptr || out16_dtype == DT_F32) YALM_CONV_T(float);
   else if (out16_dtype == DT_BF16) YALM_CONV_T(__nv_bfloat16);
   else if (out16_dtype == DT_F16) YALM_CONV_T(__half);
   else return -3;

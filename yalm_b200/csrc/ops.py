@@ -123,7 +123,7 @@ _SIGNATURES = {
     "yalm_latent_expand": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _ll, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "yalm_latent_attention_mma_usable": [_i, _i, _i],
     "yalm_latent_attention": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp,
-                              _i, _i, _vp, _i, _i, _vp],
+                              _i, _i, _i, _vp, _i, _i, _vp],
     "yalm_latent_prefill_usable": [_i, _i, _i, _i, _i, _i],
     "yalm_latent_prefill": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _ll,
                             _i, _i, _vp],
@@ -1075,11 +1075,12 @@ def latent_attention_mma_usable(dtype: torch.dtype, rank: int, hd: int) -> bool:
 def latent_attention(q: torch.Tensor, kv_step: torch.Tensor, cache: torch.Tensor, batch, slot_pos: torch.Tensor,
                      out: Optional[torch.Tensor], H: int, rank: int, hd: int, capacity: int, window: Optional[int],
                      scale: float, sink: Optional[torch.Tensor] = None, pages=None, parts=None,
-                     mma: bool = True) -> None:
+                     mma: bool = True, per_split: int = 0) -> None:
     """The absorbed form: every query q [N, H, hd] over the latent rows it sees (positions of this step from
     kv_step [N, 2, 1, hd], earlier ones from the cache), the last ``window`` positions or all; ``sink``
     float32 [H] adds exp(sink_h) to the denominator.  out [N, H, hd] (its first ``rank`` features), or with
-    ``parts`` = (part_o, part_ml, nsplit) the results of nsplit runs of keys for ``latent_expand``."""
+    ``parts`` = (part_o, part_ml, nsplit) the results of nsplit runs of ``per_split`` keys (the last takes
+    what is left) for ``latent_expand``."""
     n = batch.n_tokens
     pt, pps, npg = _pages(pages, cache, 1, hd)
     part_o, part_ml, nsplit = parts if parts is not None else (None, None, 1)
@@ -1094,7 +1095,7 @@ def latent_attention(q: torch.Tensor, kv_step: torch.Tensor, cache: torch.Tensor
     _check(lib().yalm_latent_attention(_p(q), _p(kv_step), _p(cache), _p(batch.token_seq), _p(batch.q_start),
                                        _p(batch.seq_slot), _p(slot_pos), _p(out), _p(part_o), _p(part_ml),
                                        dtype_code(q.dtype), n, H, rank, hd, capacity, int(window or 0), float(scale),
-                                       _p(sink), int(nsplit), 1 if mma else 0, pt, pps, npg, _stream()),
+                                       _p(sink), int(nsplit), int(per_split), 1 if mma else 0, pt, pps, npg, _stream()),
            "latent_attention")
 
 

@@ -2,15 +2,21 @@
 // size N and value size P:
 //   S_t = exp(a_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t,
 //   dt_t = softplus(raw_t + bias),   a_t = -exp(A_log) dt_t,
-// B and C shared by the heads of a group.  Everything here is 32-bit.  Two kernels:
+// B and C shared by the heads of a group.  Everything here is 32-bit.  Three kernels:
 //
-//  * ssd_scan: a block of four warps owns SS_COLS = 32 value columns of one (sequence, head).  The
-//    columns of S are independent; a group of eight lanes owns two of them, a lane RPT rows of
-//    those, in packed pairs, so that a token costs a lane 2 RPT updates and 2 RPT multiply-adds
-//    (half as many instructions) and the sums over the eight lanes are formed for SS_TOK tokens at
-//    once.  Tokens (B | C | the block's x) come through a three-stage cp.async ring; the steps dt
-//    and decays of a group are formed one stage ahead.  The update is S + (exp(a) - 1) S + dt B x:
-//    exp(a) - 1 as expm1, so that a decay close to one is not rounded to a float near one each time.
+//  * ssd_scan: a block owns SS_COLS = 32 value columns of one (sequence, head).  The columns of S are
+//    independent; 16 lanes own SS_CPL = 4 of them, a lane 4 K4 rows of those, in packed pairs (two FP32
+//    operations per instruction).  Four warps compute; a fifth feeds them: it brings the tokens (B | C |
+//    the block's x) through a three-stage cp.async ring of SS_TOK and turns their raw steps into dt and
+//    decays.  The sums over the 16 lanes are formed for SS_RUN tokens at once.  Runs of SS_RUN whole
+//    tokens whose decays multiply to no less than exp(-SS_SPAN) go without a decay per element: with
+//    A_t = exp(a_first + .. + a_t) and T_t = S_t / A_t,
+//        T_t = T_(t-1) + B_t (dt_t / A_t) x_t^T,   y_t = A_t T_t^T C_t,
+//    two multiply-adds per element and token, and S = T + expm1(log A) T at the run's end.  Other tokens
+//    take S + (exp(a) - 1) S + dt B x.  exp(a) - 1 is expm1 in both, so that a decay close to one is not
+//    rounded to a float near one each time.
+//  * ssd_step: the same for steps of one token per sequence (bound by the state's bytes): a warp per
+//    eight columns, the 32 lanes along a column's rows.
 //  * gated_group_norm: y silu(z), every one of `groups` equal parts of a row over its own root mean
 //    square, times a weight per feature, into the storage type.
 //
@@ -20,7 +26,8 @@
 
 namespace yalm {
 
-constexpr int SS_COLS = 32, SS_TOK = 16, SS_STAGES = 3;
+constexpr int SS_TOK = 16, SS_STAGES = 3, SS_RUN = 8, SS_CPL = 4, SS_COLS = 8 * SS_CPL;
+constexpr float SS_SPAN = 16.f;
 
 typedef unsigned long long f2;                           // two packed floats
 __device__ __forceinline__ f2 pack_f2(float lo, float hi) {
@@ -62,79 +69,100 @@ struct SsdArgs {
   int H, G, P, N;
 };
 
-// RPT rows per lane (8 RPT >= N); VEC: N, P and the pointers allow 16-byte accesses
-template <int RPT, bool VEC>
-__global__ void __launch_bounds__(128)
+__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+// K4: groups of four rows per lane (64 K4 >= N); VEC: N, P and the pointers allow 16-byte accesses
+template <int K4, bool VEC>
+__global__ void __launch_bounds__(160)
 ssd_scan_kernel(SsdArgs a) {
   pdl_launch_dependents();
-  constexpr int NP = 8 * RPT;                            // rows, padded
+  constexpr int NP = 64 * K4;                            // rows, padded
   constexpr int PER_TOK = 2 * NP + SS_COLS;              // B, C, then this block's x columns
-  constexpr int K4 = RPT / 4;
   extern __shared__ __align__(16) float ss_stage[];      // [SS_STAGES][SS_TOK][PER_TOK]
-  __shared__ float dt_s[SS_STAGES][SS_TOK], am1_s[SS_STAGES][SS_TOK];
+  // per token: exp(a) - 1, dt, and for whole runs A_t and dt / A_t
+  __shared__ __align__(16) float4 step_s[SS_STAGES][SS_TOK];
+  __shared__ float2 run_s[SS_STAGES][SS_TOK / SS_RUN];   // a run's sum of a, expm1 of it
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * SS_COLS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int sub = lane & 7, lc = warp * 8 + (lane >> 3) * 2;       // the lane's rows; its two columns in the block
   const int slot = a.seq_slot[b];
   const int t0 = a.q_start[b], t1 = a.q_start[b + 1];
-  const int N = a.N, P = a.P, inner = a.H * P, row = inner + 2 * a.G * N;
-  const int g = h / (a.H / a.G);
-  const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h], skip = a.d_skip[h];
+  const int N = a.N, P = a.P, inner = a.H * P;
   // rows beyond N and columns beyond P: never copied over, zero for ever
   if (N < NP || c0 + SS_COLS > P) {
     for (int i = threadIdx.x; i < SS_STAGES * SS_TOK * PER_TOK; i += blockDim.x) ss_stage[i] = 0.f;
     __syncthreads();
   }
   pdl_wait();
-  const int cols = min(SS_COLS, P - c0);
   const int n_groups = (t1 - t0 + SS_TOK - 1) / SS_TOK;
-  constexpr int W = VEC ? 4 : 1;
-  const int per = (2 * N + cols) / W;                    // copies per token
-  auto issue = [&](int gi) {
-    if (gi < n_groups) {
-      const int base = t0 + gi * SS_TOK;
-      const int nt = min(SS_TOK, t1 - base);
-      float* dst = ss_stage + (size_t)(gi % SS_STAGES) * SS_TOK * PER_TOK;
-      for (int e = threadIdx.x; e < per; e += blockDim.x) {
-        const int f = e * W;
-        int so, d;
-        if (f < N) { so = inner + g * N + f; d = f; }
-        else if (f < 2 * N) { so = inner + (a.G + g) * N + (f - N); d = NP + (f - N); }
-        else { so = h * P + c0 + (f - 2 * N); d = 2 * NP + (f - 2 * N); }
-        const float* src = a.act + (size_t)base * row + so;
-        for (int tt = 0; tt < nt; ++tt) ss_copy<4 * W>(dst + tt * PER_TOK + d, src + (size_t)tt * row);
+  if (warp == 4) {                                       // the warp that feeds the others
+    const int row = inner + 2 * a.G * N, g = h / (a.H / a.G);
+    const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h];
+    constexpr int W = VEC ? 4 : 1;
+    const int per = (2 * N + min(SS_COLS, P - c0)) / W;  // copies per token
+    auto issue = [&](int gi) {
+      if (gi < n_groups) {
+        const int base = t0 + gi * SS_TOK;
+        const int nt = min(SS_TOK, t1 - base);
+        float* dst = ss_stage + (size_t)(gi % SS_STAGES) * SS_TOK * PER_TOK;
+        for (int e = lane; e < per; e += 32) {
+          const int f = e * W;
+          int so, d;
+          if (f < N) { so = inner + g * N + f; d = f; }
+          else if (f < 2 * N) { so = inner + (a.G + g) * N + (f - N); d = NP + (f - N); }
+          else { so = h * P + c0 + (f - 2 * N); d = 2 * NP + (f - 2 * N); }
+          const float* src = a.act + (size_t)base * row + so;
+          for (int tt = 0; tt < nt; ++tt) ss_copy<4 * W>(dst + tt * PER_TOK + d, src + (size_t)tt * row);
+        }
       }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    auto load_dt = [&](int gi) {
+      const int t = t0 + gi * SS_TOK + lane;
+      return (lane < SS_TOK && t < t1) ? sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) : 0.f;
+    };
+    auto put_dt = [&](int gi, float raw) {
+      const float dt = softplus(raw + bias);
+      const float la = neg_a * dt;
+      float cum = la;                                    // the run's inclusive sum
+#pragma unroll
+      for (int o = 1; o < SS_RUN; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, cum, o, SS_RUN);
+        if ((lane & (SS_RUN - 1)) >= o) cum += v;
+      }
+      if (lane < SS_TOK) {
+        const float A = expf(cum);
+        step_s[gi % SS_STAGES][lane] = make_float4(expm1f(la), dt, A, dt / A);     // dt / A is read for short spans only
+        if ((lane & (SS_RUN - 1)) == SS_RUN - 1) run_s[gi % SS_STAGES][lane / SS_RUN] = make_float2(cum, expm1f(cum));
+      }
+    };
+    float raw0 = load_dt(0), raw1 = load_dt(1);
+    issue(0);
+    issue(1);
+    put_dt(0, raw0);
+    put_dt(1, raw1);
+    float raw = load_dt(2);
+    for (int gi = 0; gi < n_groups; ++gi) {
+      asm volatile("cp.async.wait_group %0;" ::"n"(SS_STAGES - 2) : "memory");
+      __syncthreads();                                   // stage gi has landed; stage gi - 1 is no longer read
+      issue(gi + 2);
+      put_dt(gi + 2, raw);
+      raw = load_dt(gi + 3);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  // a group's raw steps are loaded by threads 0 .. SS_TOK - 1 when its copies are issued, and turned into
-  // dt and exp(a) - 1 one group later
-  auto load_dt = [&](int gi) {
-    const int t = t0 + gi * SS_TOK + threadIdx.x;
-    return (threadIdx.x < SS_TOK && t < t1) ? sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) : 0.f;
-  };
-  auto put_dt = [&](int gi, float raw) {
-    if (threadIdx.x < SS_TOK) {
-      const float z = raw + bias;
-      const float dt = z > 20.f ? z : log1pf(expf(z));
-      dt_s[gi % SS_STAGES][threadIdx.x] = dt;
-      am1_s[gi % SS_STAGES][threadIdx.x] = expm1f(neg_a * dt);
-    }
-  };
-  issue(0);
-  issue(1);
-  put_dt(0, load_dt(0));
-  float raw_next = load_dt(1);
-  // the state: rows 32 k + 4 sub + j of the lane's two columns, in packed pairs
-  f2 S[2][RPT / 2];
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    return;
+  }
+  const int sub = lane & 15, lc = (warp * 2 + (lane >> 4)) * SS_CPL;       // the lane's rows; its first column in the block
+  const float skip = a.d_skip[h];
+  // the state: rows 64 k + 4 sub + j of the lane's columns, in packed pairs
+  f2 S[SS_CPL][2 * K4];
   float* st = a.state + ((size_t)slot * a.H + h) * P * N;
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < SS_CPL; ++c) {
     const int col = c0 + lc + c;
-    float* sc = st + (size_t)col * N;
+    const float* sc = st + (size_t)col * N;
 #pragma unroll
     for (int k = 0; k < K4; ++k) {
-      const int i = 32 * k + 4 * sub;
+      const int i = 64 * k + 4 * sub;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (col < P) {
         if constexpr (VEC) {
@@ -151,69 +179,104 @@ ssd_scan_kernel(SsdArgs a) {
     }
   }
   for (int gi = 0; gi < n_groups; ++gi) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(SS_STAGES - 2) : "memory");
-    __syncthreads();                                     // stage gi has landed; stage gi - 1 is no longer read
-    issue(gi + 2);
-    put_dt(gi + 1, raw_next);                            // read after the next barrier
-    raw_next = load_dt(gi + 2);
+    __syncthreads();
     const int base = t0 + gi * SS_TOK;
     const int nt = min(SS_TOK, t1 - base);
     const float* sg = ss_stage + (size_t)(gi % SS_STAGES) * SS_TOK * PER_TOK;
-    const float* dts = dt_s[gi % SS_STAGES];
-    const float* ams = am1_s[gi % SS_STAGES];
-    float o[SS_TOK * 2];
+    const float4* steps = step_s[gi % SS_STAGES];
+#pragma unroll 1
+    for (int r = 0; r < SS_TOK / SS_RUN; ++r) {
+      const int first = r * SS_RUN;
+      if (first >= nt) break;
+      const float2 run = run_s[gi % SS_STAGES][r];
+      float o[SS_RUN * SS_CPL];
+      if (nt >= first + SS_RUN && run.x >= -SS_SPAN) {
 #pragma unroll
-    for (int tt = 0; tt < SS_TOK; ++tt) {
-      o[2 * tt] = o[2 * tt + 1] = 0.f;
-      if (tt < nt) {
-        const float* p = sg + tt * PER_TOK;
-        const float2 x = *reinterpret_cast<const float2*>(p + 2 * NP + lc);
-        const float dt = dts[tt], am1 = ams[tt];
-        const f2 am = pack_f2(am1, am1);
-        const f2 xd0 = pack_f2(dt * x.x, dt * x.x), xd1 = pack_f2(dt * x.y, dt * x.y);
-        f2 o0 = 0ull, o1 = 0ull;                         // two zeros
+        for (int tt = 0; tt < SS_RUN; ++tt) {
+          const float* p = sg + (first + tt) * PER_TOK;
+          const float4 sv = steps[first + tt];
+          const float4 xv = *reinterpret_cast<const float4*>(p + 2 * NP + lc);
+          const float x[SS_CPL] = {sv.w * xv.x, sv.w * xv.y, sv.w * xv.z, sv.w * xv.w};
+          f2 oc[SS_CPL];
 #pragma unroll
-        for (int k = 0; k < K4; ++k) {
-          const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(p + 32 * k + 4 * sub);
-          const ulonglong2 C = *reinterpret_cast<const ulonglong2*>(p + NP + 32 * k + 4 * sub);
-          S[0][2 * k] = add_f2(S[0][2 * k], fma_f2(am, S[0][2 * k], mul_f2(B.x, xd0)));
-          S[1][2 * k] = add_f2(S[1][2 * k], fma_f2(am, S[1][2 * k], mul_f2(B.x, xd1)));
-          S[0][2 * k + 1] = add_f2(S[0][2 * k + 1], fma_f2(am, S[0][2 * k + 1], mul_f2(B.y, xd0)));
-          S[1][2 * k + 1] = add_f2(S[1][2 * k + 1], fma_f2(am, S[1][2 * k + 1], mul_f2(B.y, xd1)));
-          o0 = fma_f2(S[0][2 * k], C.x, o0);
-          o1 = fma_f2(S[1][2 * k], C.x, o1);
-          o0 = fma_f2(S[0][2 * k + 1], C.y, o0);
-          o1 = fma_f2(S[1][2 * k + 1], C.y, o1);
+          for (int k = 0; k < K4; ++k) {
+            const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(p + 64 * k + 4 * sub);
+            const ulonglong2 C = *reinterpret_cast<const ulonglong2*>(p + NP + 64 * k + 4 * sub);
+#pragma unroll
+            for (int c = 0; c < SS_CPL; ++c) {
+              const f2 xd = pack_f2(x[c], x[c]);
+              S[c][2 * k] = fma_f2(B.x, xd, S[c][2 * k]);
+              S[c][2 * k + 1] = fma_f2(B.y, xd, S[c][2 * k + 1]);
+              oc[c] = k == 0 ? mul_f2(S[c][0], C.x) : fma_f2(S[c][2 * k], C.x, oc[c]);
+              oc[c] = fma_f2(S[c][2 * k + 1], C.y, oc[c]);
+            }
+          }
+#pragma unroll
+          for (int c = 0; c < SS_CPL; ++c) {
+            float lo, hi;
+            unpack_f2(oc[c], lo, hi);
+            o[SS_CPL * tt + c] = sv.z * (lo + hi);
+          }
         }
-        float lo, hi;
-        unpack_f2(o0, lo, hi);
-        o[2 * tt] = lo + hi;
-        unpack_f2(o1, lo, hi);
-        o[2 * tt + 1] = lo + hi;
+        const f2 e = pack_f2(run.y, run.y);
+#pragma unroll
+        for (int c = 0; c < SS_CPL; ++c)
+#pragma unroll
+          for (int k = 0; k < 2 * K4; ++k) S[c][k] = fma_f2(e, S[c][k], S[c][k]);
+      } else {
+#pragma unroll
+        for (int tt = 0; tt < SS_RUN; ++tt) {
+#pragma unroll
+          for (int c = 0; c < SS_CPL; ++c) o[SS_CPL * tt + c] = 0.f;
+          if (first + tt < nt) {
+            const float* p = sg + (first + tt) * PER_TOK;
+            const float4 sv = steps[first + tt];
+            const f2 am = pack_f2(sv.x, sv.x);
+            const float4 xv = *reinterpret_cast<const float4*>(p + 2 * NP + lc);
+            const float x[SS_CPL] = {sv.y * xv.x, sv.y * xv.y, sv.y * xv.z, sv.y * xv.w};
+            f2 oc[SS_CPL];
+#pragma unroll
+            for (int k = 0; k < K4; ++k) {
+              const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(p + 64 * k + 4 * sub);
+              const ulonglong2 C = *reinterpret_cast<const ulonglong2*>(p + NP + 64 * k + 4 * sub);
+#pragma unroll
+              for (int c = 0; c < SS_CPL; ++c) {
+                const f2 xd = pack_f2(x[c], x[c]);
+                S[c][2 * k] = add_f2(S[c][2 * k], fma_f2(am, S[c][2 * k], mul_f2(B.x, xd)));
+                S[c][2 * k + 1] = add_f2(S[c][2 * k + 1], fma_f2(am, S[c][2 * k + 1], mul_f2(B.y, xd)));
+                oc[c] = k == 0 ? mul_f2(S[c][0], C.x) : fma_f2(S[c][2 * k], C.x, oc[c]);
+                oc[c] = fma_f2(S[c][2 * k + 1], C.y, oc[c]);
+              }
+            }
+#pragma unroll
+            for (int c = 0; c < SS_CPL; ++c) {
+              float lo, hi;
+              unpack_f2(oc[c], lo, hi);
+              o[SS_CPL * tt + c] = lo + hi;
+            }
+          }
+        }
       }
-    }
-    // the group's 2 SS_TOK outputs of these columns, each the sum of eight lanes' parts: in every round a
-    // lane hands half of its values over and adds the other half of its partner's, so that lane `sub`
-    // ends with the whole sums of values 4 s .. 4 s + 3 (two tokens), s = its bits from 4 down to 1
+      // the run's 32 outputs of these four columns (number 4 tt + c), each the sum of 16 lanes' parts: in
+      // every round a lane hands half of its values over and adds the other half of its partner's, so that
+      // lane `sub` ends with the whole sums number 2 sub and 2 sub + 1
+      static_assert(SS_RUN * SS_CPL == 32, "two outputs per lane");
 #pragma unroll
-    for (int half = SS_TOK; half >= SS_TOK / 4; half >>= 1) {
-      const int bit = half * 4 / SS_TOK;                 // lane bits 4, 2, 1
-      const bool upper = (lane & bit) != 0;
+      for (int half = 16; half >= 2; half >>= 1) {
+        const bool upper = (lane & (half >> 1)) != 0;
 #pragma unroll
-      for (int i = 0; i < half; ++i) {
-        const float send = upper ? o[i] : o[i + half];
-        const float keep = upper ? o[i + half] : o[i];
-        o[i] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+        for (int i = 0; i < half; ++i) {
+          const float send = upper ? o[i] : o[i + half];
+          const float keep = upper ? o[i + half] : o[i];
+          o[i] = keep + __shfl_xor_sync(0xffffffffu, send, half >> 1);
+        }
       }
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int tt = sub * 2 + i, col = c0 + lc;
+      const int tt = first + (sub >> 1), lcc = lc + (sub & 1) * 2, col = c0 + lcc;
       if (tt < nt && col < P) {
-        const float* x = sg + tt * PER_TOK + 2 * NP + lc;
+        const float2 x = *reinterpret_cast<const float2*>(sg + tt * PER_TOK + 2 * NP + lcc);
+        const float y0 = fmaf(skip, x.x, o[0]), y1 = fmaf(skip, x.y, o[1]);
         float* dst = a.out + (size_t)(base + tt) * inner + h * P + col;
-        const float y0 = fmaf(skip, x[0], o[2 * i]), y1 = fmaf(skip, x[1], o[2 * i + 1]);
-        if (VEC) {
+        if constexpr (VEC) {
           *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
         } else {
           dst[0] = y0;
@@ -222,15 +285,14 @@ ssd_scan_kernel(SsdArgs a) {
       }
     }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
+  for (int c = 0; c < SS_CPL; ++c) {
     const int col = c0 + lc + c;
     if (col >= P) continue;
     float* sc = st + (size_t)col * N;
 #pragma unroll
     for (int k = 0; k < K4; ++k) {
-      const int i = 32 * k + 4 * sub;
+      const int i = 64 * k + 4 * sub;
       float4 v;
       unpack_f2(S[c][2 * k], v.x, v.y);
       unpack_f2(S[c][2 * k + 1], v.z, v.w);
@@ -244,6 +306,80 @@ ssd_scan_kernel(SsdArgs a) {
       }
     }
   }
+}
+
+constexpr int SD_COLS = 8;                               // columns per warp of ssd_step
+
+// One token per sequence.  grid (column tiles of 8 SD_COLS, heads, sequences), eight warps
+template <bool VEC>
+__global__ void __launch_bounds__(256, 3)
+ssd_step_kernel(SsdArgs a) {
+  pdl_launch_dependents();
+  const int b = blockIdx.z, h = blockIdx.y;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int c0 = (blockIdx.x * 8 + warp) * SD_COLS;
+  const int slot = a.seq_slot[b], t = a.q_start[b];
+  const int N = a.N, P = a.P, inner = a.H * P;
+  if (c0 >= P) return;
+  const int g = h / (a.H / a.G);
+  float* st = a.state + ((size_t)slot * a.H + h) * P * N;
+  const float* row = a.act + (size_t)t * (inner + 2 * a.G * N);
+  pdl_wait();
+  const float dt = softplus(sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) + a.dt_bias[h]);
+  const float am1 = expm1f(-expf(a.a_log[h]) * dt);
+  float x[SD_COLS], y[SD_COLS];
+#pragma unroll
+  for (int c = 0; c < SD_COLS; ++c) {
+    x[c] = c0 + c < P ? row[h * P + c0 + c] : 0.f;
+    y[c] = 0.f;
+  }
+  constexpr int W = VEC ? 4 : 1;
+  for (int i = lane * W; i < N; i += 32 * W) {
+    float B[W], C[W], S[SD_COLS][W];
+    if constexpr (VEC) {
+#pragma unroll
+      for (int c = 0; c < SD_COLS; ++c) {
+        const float4 v = c0 + c < P ? *reinterpret_cast<const float4*>(st + (size_t)(c0 + c) * N + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        S[c][0] = v.x; S[c][1] = v.y; S[c][2] = v.z; S[c][3] = v.w;
+      }
+      const float4 u = *reinterpret_cast<const float4*>(row + inner + g * N + i);
+      const float4 w = *reinterpret_cast<const float4*>(row + inner + (a.G + g) * N + i);
+      B[0] = u.x; B[1] = u.y; B[2] = u.z; B[3] = u.w;
+      C[0] = w.x; C[1] = w.y; C[2] = w.z; C[3] = w.w;
+    } else {
+#pragma unroll
+      for (int c = 0; c < SD_COLS; ++c) S[c][0] = c0 + c < P ? st[(size_t)(c0 + c) * N + i] : 0.f;
+      B[0] = row[inner + g * N + i];
+      C[0] = row[inner + (a.G + g) * N + i];
+    }
+#pragma unroll
+    for (int c = 0; c < SD_COLS; ++c) {
+#pragma unroll
+      for (int j = 0; j < W; ++j) {
+        S[c][j] += fmaf(am1, S[c][j], B[j] * (dt * x[c]));
+        y[c] = fmaf(S[c][j], C[j], y[c]);
+      }
+      if (c0 + c < P) {
+        if constexpr (VEC) *reinterpret_cast<float4*>(st + (size_t)(c0 + c) * N + i) = make_float4(S[c][0], S[c][1], S[c][2], S[c][3]);
+        else st[(size_t)(c0 + c) * N + i] = S[c][0];
+      }
+    }
+  }
+  // eight sums over 32 lanes: three rounds leave one value per lane, two more add up the quarters
+#pragma unroll
+  for (int half = 4; half >= 1; half >>= 1) {
+    const bool upper = (lane & half) != 0;
+#pragma unroll
+    for (int i = 0; i < half; ++i) {
+      const float send = upper ? y[i] : y[i + half];
+      const float keep = upper ? y[i + half] : y[i];
+      y[i] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+    }
+  }
+  y[0] += __shfl_xor_sync(0xffffffffu, y[0], 8);
+  y[0] += __shfl_xor_sync(0xffffffffu, y[0], 16);
+  if (lane < SD_COLS && c0 + lane < P)
+    a.out[(size_t)t * inner + h * P + c0 + lane] = fmaf(a.d_skip[h], row[h * P + c0 + lane], y[0]);
 }
 
 // grid (tokens, groups); y [tokens][inner]; z slices [z_n][tokens][z_row]; out [tokens][inner]
@@ -313,29 +449,35 @@ extern "C" int yalm_ssd_scan(const float* act, const float* dt, int dt_n, long l
   if (H <= 0 || G <= 0 || H % G || P <= 0 || N <= 0 || N > 256) return -2;
   if (n_seqs > 65535 || H > 65535) return -4;
   const SsdArgs a = {act, dt + col0, dt_n, dt_row, dt_stride, dt_bias, a_log, d_skip, q_start, seq_slot, state, out, H, G, P, N};
-  const dim3 grid((P + SS_COLS - 1) / SS_COLS, H, n_seqs), block(128);
   const bool vec = N % 4 == 0 && P % 4 == 0 && ((((uintptr_t)act) | ((uintptr_t)state) | ((uintptr_t)out)) & 15) == 0;
-#define YALM_SSD1(R, V)                                                                                       \
+  if (n_tokens == n_seqs) {                              // every sequence brings one token
+    const dim3 sgrid((P + 8 * SD_COLS - 1) / (8 * SD_COLS), H, n_seqs), sblock(256);
+    if (vec) launch_pdl(ssd_step_kernel<true>, sgrid, sblock, 0, stream, a);
+    else launch_pdl(ssd_step_kernel<false>, sgrid, sblock, 0, stream, a);
+    YALM_LAUNCH_CHECK();
+    return 0;
+  }
+  const dim3 grid((P + SS_COLS - 1) / SS_COLS, H, n_seqs), block(160);
+#define YALM_SSD1(K, V)                                                                                       \
   do {                                                                                                        \
-    const size_t smem = (size_t)SS_STAGES * SS_TOK * (2 * 8 * R + SS_COLS) * sizeof(float);                   \
+    const size_t smem = (size_t)SS_STAGES * SS_TOK * (2 * 64 * K + SS_COLS) * sizeof(float);                  \
     static bool set = false;                                                                                  \
     if (!set && smem > 40 * 1024) {                                                                           \
-      cudaError_t e = cudaFuncSetAttribute(ssd_scan_kernel<R, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaError_t e = cudaFuncSetAttribute(ssd_scan_kernel<K, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                            (int)smem);                                                        \
       if (e != cudaSuccess) return (int)e;                                                                    \
       set = true;                                                                                             \
     }                                                                                                         \
-    launch_pdl(ssd_scan_kernel<R, V>, grid, block, smem, stream, a);                                          \
+    launch_pdl(ssd_scan_kernel<K, V>, grid, block, smem, stream, a);                                          \
   } while (0)
-#define YALM_SSD(R)              \
+#define YALM_SSD(K)              \
   do {                           \
-    if (vec) YALM_SSD1(R, true); \
-    else YALM_SSD1(R, false);    \
+    if (vec) YALM_SSD1(K, true); \
+    else YALM_SSD1(K, false);    \
   } while (0)
-  if (N <= 32) YALM_SSD(4);
-  else if (N <= 64) YALM_SSD(8);
-  else if (N <= 128) YALM_SSD(16);
-  else YALM_SSD(32);
+  if (N <= 64) YALM_SSD(1);
+  else if (N <= 128) YALM_SSD(2);
+  else YALM_SSD(4);
 #undef YALM_SSD
 #undef YALM_SSD1
   YALM_LAUNCH_CHECK();

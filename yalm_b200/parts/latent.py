@@ -143,17 +143,21 @@ class LatentAttention:
         per_pair = self.dim + self.rd + self.vdim if all(p == 0 for p in past) else 2 * self.rank + self.rd
         return lin + 2.0 * H * per_pair * pairs
 
-    def decode_splits(self, batch, mma: bool) -> int:
-        """Runs of keys per query: as many as let the grid fill the SMs, with at least two tiles of 64 keys
-        each (by the step's bound: a captured decode step keeps its plan)."""
+    def decode_splits(self, batch, mma: bool):
+        """(runs of keys per query, keys per run): runs as long as let the runs of all queries fill the SMs'
+        block slots (two each), two tiles of 32 keys at least.  Runs are of one size, so that a batch's
+        long sequences get more blocks than its short ones; lengths are counted as they will be when the
+        longest reaches the step's bound (a captured decode step keeps its plan)."""
         if batch.n_tokens > ops.LATENT_FEW_TOKENS or not (mma or batch.is_decode):
-            return 1
+            return 1, 0
         bound = max(1, batch.ctx_bound)
-        visible = min(bound, self.window) if self.window else bound
-        tiles = -(-visible // 64)
-        blocks = batch.n_tokens * -(-self.H // (16 if mma else 4))
-        room = (1 if mma and self.hd > 256 else 2) * self.rt.sm_count
-        return max(1, min(tiles // 2, room // blocks, ops.LATENT_MAX_SPLIT))
+        slack = max(0, bound - max(p + q for p, q in zip(batch.past, batch.q_lens)))
+        seen = lambda n: -(-(min(n, self.window) if self.window else n) // 32)
+        total = sum(q * seen(p + q + slack) for p, q in zip(batch.past, batch.q_lens))
+        groups = -(-self.H // (16 if mma else 4))
+        most = seen(bound)
+        per = max(2, -(-total * groups // (2 * self.rt.sm_count)), -(-most // ops.LATENT_MAX_SPLIT))
+        return -(-most // per), per * 32
 
     def forward(self, h, batch, stream, view, shared: bool = False):
         rt, H, hd, rank = self.rt, self.H, self.hd, self.rank
@@ -189,7 +193,7 @@ class LatentAttention:
             q = rt.buffer("latent_q_abs", (n, H * hd), rt.dtype)
             ops.latent_absorb_q(z, S, self.w_uk, self.freq, batch, view.slot_pos, q, H, self.dim, self.rd, rank, hd, **rot)
             mma = rt.attention != "simt" and ops.latent_attention_mma_usable(rt.dtype, rank, hd)
-            nsplit = self.decode_splits(batch, mma)
+            nsplit, per = self.decode_splits(batch, mma)
             o_lat = parts = None
             if nsplit > 1:
                 parts = (rt.buffer("latent_part_o", (n, H, nsplit, rank), torch.float32),
@@ -197,7 +201,8 @@ class LatentAttention:
             else:
                 o_lat = rt.buffer("latent_mixed", (n, H * hd), rt.dtype)
             ops.latent_attention(q, kv_step, view.k, batch, view.slot_pos, o_lat, H, rank, hd, view.capacity,
-                                 self.window, self.scale, sink=self.sink, pages=view.pages, parts=parts, mma=mma)
+                                 self.window, self.scale, sink=self.sink, pages=view.pages, parts=parts,
+                                 mma=mma, per_split=per)
             ops.latent_expand(o_lat, self.w_uv, z if self.gate else None, S, o, H, rank, self.vdim, hd, parts=parts, **gate)
         stream.add_linear(o, self.w_o)
         if late_write:
