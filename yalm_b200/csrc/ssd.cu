@@ -12,9 +12,10 @@
 //    tokens whose decays multiply to no less than exp(-SS_SPAN) go without a decay per element: with
 //    A_t = exp(a_first + .. + a_t) and T_t = S_t / A_t,
 //        T_t = T_(t-1) + B_t (dt_t / A_t) x_t^T,   y_t = A_t T_t^T C_t,
-//    two multiply-adds per element and token, and S = T + expm1(log A) T at the run's end.  Other tokens
-//    take S + (exp(a) - 1) S + dt B x.  exp(a) - 1 is expm1 in both, so that a decay close to one is not
-//    rounded to a float near one each time.
+//    two multiply-adds per element and token, and S = A T at the run's end.  Other tokens take
+//    exp(a) S + dt B x.  A decay above one half is applied as S + (exp(a) - 1) S with exp(a) - 1 = expm1(a),
+//    so that one close to one is not rounded to a float near one each time; a smaller one as it is, so
+//    that what it leaves is not the difference of two nearly equal numbers.
 //  * ssd_step: the same for steps of one token per sequence (bound by the state's bytes): a warp per
 //    eight columns, the 32 lanes along a column's rows.
 //  * gated_group_norm: y silu(z), every one of `groups` equal parts of a row over its own root mean
@@ -46,12 +47,6 @@ __device__ __forceinline__ f2 mul_f2(f2 a, f2 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
-__device__ __forceinline__ f2 add_f2(f2 a, f2 b) {
-  f2 r;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-
 template <int BYTES>
 __device__ __forceinline__ void ss_copy(float* dst, const float* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
@@ -71,6 +66,11 @@ struct SsdArgs {
 
 __device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
+// A decay exp(a), a <= 0, as it is applied: S <- coef S + keep S, with keep 1 where coef = exp(a) - 1 (its sign
+// bit is set, also for a = -0) and 0 where coef = exp(a)
+__device__ __forceinline__ float decay_coef(float a) { return a > -0.69f ? expm1f(a) : expf(a); }
+__device__ __forceinline__ float decay_keep(float coef) { return signbit(coef) ? 1.f : 0.f; }
+
 // K4: groups of four rows per lane (64 K4 >= N); VEC: N, P and the pointers allow 16-byte accesses
 template <int K4, bool VEC>
 __global__ void __launch_bounds__(160)
@@ -79,9 +79,9 @@ ssd_scan_kernel(SsdArgs a) {
   constexpr int NP = 64 * K4;                            // rows, padded
   constexpr int PER_TOK = 2 * NP + SS_COLS;              // B, C, then this block's x columns
   extern __shared__ __align__(16) float ss_stage[];      // [SS_STAGES][SS_TOK][PER_TOK]
-  // per token: exp(a) - 1, dt, and for whole runs A_t and dt / A_t
+  // per token: the decay's coefficient, dt, and for whole runs A_t and dt / A_t
   __shared__ __align__(16) float4 step_s[SS_STAGES][SS_TOK];
-  __shared__ float2 run_s[SS_STAGES][SS_TOK / SS_RUN];   // a run's sum of a, expm1 of it
+  __shared__ float2 run_s[SS_STAGES][SS_TOK / SS_RUN];   // a run's sum of a, its decay's coefficient
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * SS_COLS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int slot = a.seq_slot[b];
@@ -131,8 +131,8 @@ ssd_scan_kernel(SsdArgs a) {
       }
       if (lane < SS_TOK) {
         const float A = expf(cum);
-        step_s[gi % SS_STAGES][lane] = make_float4(expm1f(la), dt, A, dt / A);     // dt / A is read for short spans only
-        if ((lane & (SS_RUN - 1)) == SS_RUN - 1) run_s[gi % SS_STAGES][lane / SS_RUN] = make_float2(cum, expm1f(cum));
+        step_s[gi % SS_STAGES][lane] = make_float4(decay_coef(la), dt, A, dt / A);     // dt / A is read for short spans only
+        if ((lane & (SS_RUN - 1)) == SS_RUN - 1) run_s[gi % SS_STAGES][lane / SS_RUN] = make_float2(cum, decay_coef(cum));
       }
     };
     float raw0 = load_dt(0), raw1 = load_dt(1);
@@ -218,11 +218,12 @@ ssd_scan_kernel(SsdArgs a) {
             o[SS_CPL * tt + c] = sv.z * (lo + hi);
           }
         }
-        const f2 e = pack_f2(run.y, run.y);
+        const float keep = decay_keep(run.y);
+        const f2 e = pack_f2(run.y, run.y), kp = pack_f2(keep, keep);
 #pragma unroll
         for (int c = 0; c < SS_CPL; ++c)
 #pragma unroll
-          for (int k = 0; k < 2 * K4; ++k) S[c][k] = fma_f2(e, S[c][k], S[c][k]);
+          for (int k = 0; k < 2 * K4; ++k) S[c][k] = fma_f2(e, S[c][k], mul_f2(kp, S[c][k]));
       } else {
 #pragma unroll
         for (int tt = 0; tt < SS_RUN; ++tt) {
@@ -231,7 +232,8 @@ ssd_scan_kernel(SsdArgs a) {
           if (first + tt < nt) {
             const float* p = sg + (first + tt) * PER_TOK;
             const float4 sv = steps[first + tt];
-            const f2 am = pack_f2(sv.x, sv.x);
+            const float keep = decay_keep(sv.x);
+            const f2 am = pack_f2(sv.x, sv.x), kp = pack_f2(keep, keep);
             const float4 xv = *reinterpret_cast<const float4*>(p + 2 * NP + lc);
             const float x[SS_CPL] = {sv.y * xv.x, sv.y * xv.y, sv.y * xv.z, sv.y * xv.w};
             f2 oc[SS_CPL];
@@ -242,8 +244,8 @@ ssd_scan_kernel(SsdArgs a) {
 #pragma unroll
               for (int c = 0; c < SS_CPL; ++c) {
                 const f2 xd = pack_f2(x[c], x[c]);
-                S[c][2 * k] = add_f2(S[c][2 * k], fma_f2(am, S[c][2 * k], mul_f2(B.x, xd)));
-                S[c][2 * k + 1] = add_f2(S[c][2 * k + 1], fma_f2(am, S[c][2 * k + 1], mul_f2(B.y, xd)));
+                S[c][2 * k] = fma_f2(kp, S[c][2 * k], fma_f2(am, S[c][2 * k], mul_f2(B.x, xd)));
+                S[c][2 * k + 1] = fma_f2(kp, S[c][2 * k + 1], fma_f2(am, S[c][2 * k + 1], mul_f2(B.y, xd)));
                 oc[c] = k == 0 ? mul_f2(S[c][0], C.x) : fma_f2(S[c][2 * k], C.x, oc[c]);
                 oc[c] = fma_f2(S[c][2 * k + 1], C.y, oc[c]);
               }
@@ -326,7 +328,7 @@ ssd_step_kernel(SsdArgs a) {
   const float* row = a.act + (size_t)t * (inner + 2 * a.G * N);
   pdl_wait();
   const float dt = softplus(sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) + a.dt_bias[h]);
-  const float am1 = expm1f(-expf(a.a_log[h]) * dt);
+  const float coef = decay_coef(-expf(a.a_log[h]) * dt), keep = decay_keep(coef);
   float x[SD_COLS], y[SD_COLS];
 #pragma unroll
   for (int c = 0; c < SD_COLS; ++c) {
@@ -356,7 +358,7 @@ ssd_step_kernel(SsdArgs a) {
     for (int c = 0; c < SD_COLS; ++c) {
 #pragma unroll
       for (int j = 0; j < W; ++j) {
-        S[c][j] += fmaf(am1, S[c][j], B[j] * (dt * x[c]));
+        S[c][j] = fmaf(keep, S[c][j], fmaf(coef, S[c][j], B[j] * (dt * x[c])));
         y[c] = fmaf(S[c][j], C[j], y[c]);
       }
       if (c0 + c < P) {
