@@ -393,11 +393,11 @@ struct PromptArgs {
   int H, dim, rd, vdim, rank, hd, window;
   float scale_log2;
 };
-constexpr int LP_BQ = 64, LP_BK = 64;
+constexpr int LP_BQ = 64, LP_BK = 32;
 
 // NV: 16-column groups of the values (vdim <= 16 NV)
 template <typename T, int NV>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, NV <= 8 ? 3 : 1)
 attn_latent_prefill_kernel(PromptArgs a) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) uint8_t lp_smem[];
@@ -425,13 +425,14 @@ attn_latent_prefill_kernel(PromptArgs a) {
   const T* q = reinterpret_cast<const T*>(a.q);
   const T* kv = reinterpret_cast<const T*>(a.kv);
   const T* rows = reinterpret_cast<const T*>(a.kv_step);
-  const int cr = threadIdx.x >> 1, ch = threadIdx.x & 1;           // a copied row and its odd or even pieces
+  constexpr int TPR = 128 / LP_BK;                                 // threads that copy a key's row
+  const int cr = threadIdx.x / TPR, ch = threadIdx.x % TPR;
   const int kvd = a.dim + a.vdim;
   {
-    const int row = p_first + cr;
+    const int r = threadIdx.x >> 1, row = p_first + r;
     const bool on = row < ql;
     const T* src = q + ((size_t)(qs + (on ? row : 0)) * a.H + h) * qd;
-    for (int c = ch; c < qd / 8; c += 2) cp16(qt + cr * ldk + c * 8, src + c * 8, on ? 16 : 0);
+    for (int c = threadIdx.x & 1; c < qd / 8; c += 2) cp16(qt + r * ldk + c * 8, src + c * 8, on ? 16 : 0);
   }
   auto issue = [&](int kb) {
     const int key = j_lo + kb * LP_BK + cr;
@@ -442,9 +443,9 @@ attn_latent_prefill_kernel(PromptArgs a) {
     T* kd = kt + (size_t)(kb & 1) * LP_BK * ldk + cr * ldk;
     T* vd = vt + (size_t)(kb & 1) * LP_BK * LDV + cr * LDV;
     const uint32_t bytes = on ? 16 : 0;
-    for (int c = ch; c < a.dim / 8; c += 2) cp16(kd + c * 8, src + c * 8, bytes);
-    for (int c = ch; c < a.rd / 8; c += 2) cp16(kd + a.dim + c * 8, rope + c * 8, bytes);
-    for (int c = ch; c < a.vdim / 8; c += 2) cp16(vd + c * 8, src + a.dim + c * 8, bytes);
+    for (int c = ch; c < a.dim / 8; c += TPR) cp16(kd + c * 8, src + c * 8, bytes);
+    for (int c = ch; c < a.rd / 8; c += TPR) cp16(kd + a.dim + c * 8, rope + c * 8, bytes);
+    for (int c = ch; c < a.vdim / 8; c += TPR) cp16(vd + c * 8, src + a.dim + c * 8, bytes);
     cp_commit();
   };
   float o[2 * NV][4];
@@ -469,16 +470,16 @@ attn_latent_prefill_kernel(PromptArgs a) {
     __syncthreads();
     const T* ks = kt + (size_t)(kb & 1) * LP_BK * ldk;
     const T* vs = vt + (size_t)(kb & 1) * LP_BK * LDV;
-    float s[8][4];
+    float s[LP_BK / 8][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+    for (int i = 0; i < LP_BK / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
     const uint32_t kaddr = smem_u32(ks + ((mi >> 1) * 8 + mr) * ldk + (mi & 1) * 8);
 #pragma unroll 2
     for (int kk = 0; kk < nk; ++kk) {
       uint32_t qf[4];
       ldsm_x4(qf, qaddr + kk * 32);
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
+      for (int n2 = 0; n2 < LP_BK / 16; ++n2) {
         uint32_t r[4];
         ldsm_x4(r, kaddr + (uint32_t)(n2 * 16 * ldk + kk * 16) * 2);
         mma16<T>(s[2 * n2], qf, r[0], r[1]);
@@ -491,7 +492,7 @@ attn_latent_prefill_kernel(PromptArgs a) {
     const int lo0 = first_visible(r0, a.window), lo1 = first_visible(r1, a.window);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt)
+    for (int nt = 0; nt < LP_BK / 8; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int rr = e >> 1;
@@ -518,7 +519,7 @@ attn_latent_prefill_kernel(PromptArgs a) {
       }
       float sum = 0.f;
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
+      for (int nt = 0; nt < LP_BK / 8; ++nt)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const float p = exp2f(s[nt][2 * rr + e] - sub);
@@ -529,7 +530,7 @@ attn_latent_prefill_kernel(PromptArgs a) {
     }
     const uint32_t vaddr = smem_u32(vs + ((mi & 1) * 8 + mr) * LDV + (mi >> 1) * 8);
 #pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
+    for (int kk = 0; kk < LP_BK / 16; ++kk) {
       uint32_t hi[4], mid[4], low[4];
       three_terms<T>(s[2 * kk][0], s[2 * kk][1], hi[0], mid[0], low[0]);
       three_terms<T>(s[2 * kk][2], s[2 * kk][3], hi[1], mid[1], low[1]);
