@@ -18,6 +18,7 @@ equal share one *group*, which has storage of its own:
   sequence has one block of its own, ``K, V : [entries, slots, kv_heads, capacity,
   head_dim]``, no table: the decode attention streams from that layout 5 to 20 %
   faster (batch 8 to 64 at 7B sizes).
+  A need with ``value_dim`` keeps values of that size beside keys of ``head_dim``.
   A need with ``values=False`` has one plane: its rows serve as keys and as values (a cached
   latent), and the view's ``v`` is its ``k``.
 * ``state`` groups hold ``[entries, slots, *shape]`` of fixed size per
@@ -57,13 +58,19 @@ class CacheNeed:
     window: Optional[int] = None               # kv: keep only the last `window` positions
     every: int = 1                             # kv: one row per `every` positions (row r: block r)
     values: bool = True                        # kv: False when a row serves as key AND value (one plane)
+    value_dim: Optional[int] = None            # kv: the values' size where it is not head_dim
     state_shape: Tuple[int, ...] = ()          # state: per-sequence shape
     state_dtype: torch.dtype = torch.float32
 
     def group_key(self, context: int):
         if self.kind == "kv":
-            return ("kv", self.kv_heads, self.head_dim, self.capacity(context), self.every, self.values)
+            return ("kv", self.kv_heads, self.head_dim, self.capacity(context), self.every, self.values,
+                    self.value_size)
         return ("state", tuple(self.state_shape), self.state_dtype)
+
+    @property
+    def value_size(self) -> int:
+        return self.value_dim or self.head_dim
 
     def capacity(self, context: int) -> int:
         if self.every > 1:
@@ -156,14 +163,10 @@ class Cache:
                 n_pages = _pool_pages(need, n_slots, context, max_tokens)
                 g["capacity"] = cap
                 if n_pages == 0:                                   # one block per sequence
-                    shape = (n, n_slots, need.kv_heads, cap, need.head_dim)
-                    g["k"] = torch.zeros(shape, dtype=dtype, device=self.device)
-                    g["v"] = torch.zeros(shape, dtype=dtype, device=self.device) if need.values else g["k"]
+                    self._planes(g, need, (n, n_slots, need.kv_heads, cap))
                     continue
-                shape = (n, need.kv_heads, n_pages, PAGE, need.head_dim)
                 g["pages_per_slot"] = -(-cap // PAGE)
-                g["k"] = torch.zeros(shape, dtype=dtype, device=self.device)
-                g["v"] = torch.zeros(shape, dtype=dtype, device=self.device) if need.values else g["k"]
+                self._planes(g, need, (n, need.kv_heads, n_pages, PAGE))
                 g["pool"] = SlotAllocator(n_pages, what="page")
                 g["held"] = [[] for _ in range(n_slots)]           # a slot's pages, in row order
                 table = torch.zeros((n_slots, g["pages_per_slot"]), dtype=torch.int32)
@@ -176,6 +179,10 @@ class Cache:
                                          dtype=need.state_dtype, device=self.device)
             else:
                 raise ValueError(f"unknown cache kind {need.kind!r}")
+
+    def _planes(self, g: dict, need: CacheNeed, shape: Tuple[int, ...]) -> None:
+        g["k"] = torch.zeros(shape + (need.head_dim,), dtype=self.dtype, device=self.device)
+        g["v"] = torch.zeros(shape + (need.value_size,), dtype=self.dtype, device=self.device) if need.values else g["k"]
 
     # -- sizes ---------------------------------------------------------------
     def bytes(self) -> int:
@@ -195,7 +202,7 @@ class Cache:
             if need.kind == "kv":
                 pages = _pool_pages(need, n_slots, context, max_tokens)
                 rows = pages * PAGE if pages else n_slots * need.capacity(context)
-                total += (2 if need.values else 1) * rows * need.kv_heads * need.head_dim * esz
+                total += rows * need.kv_heads * (need.head_dim + (need.value_size if need.values else 0)) * esz
             else:
                 n = 1
                 for s in need.state_shape:

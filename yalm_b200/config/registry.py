@@ -16,6 +16,7 @@ from .nekotar import NekotarConfig
 from .rudazen import RudazenConfig
 from .samulorn import SamulornConfig
 from .saralix import SaralixConfig
+from .tetodra import TetodraConfig
 
 _ARCHITECTURES: Dict[str, Any] = {}
 
@@ -58,3 +59,4 @@ register_architecture("Rudazen", RudazenConfig)
 register_architecture("Nekotar", NekotarConfig)
 register_architecture("Samulorn", SamulornConfig)
 register_architecture("Saralix", SaralixConfig)
+register_architecture("Tetodra", TetodraConfig)

@@ -366,9 +366,32 @@ int yalm_latent_prefill(const void* q, const void* kv, const void* kv_step, cons
 
 // ---- ssd.cu: a state-space recurrence with one decay per head ------------------------------------
 int yalm_ssd_scan(const float* act, const float* dt, int dt_n, long long dt_stride, int dt_row, int col0,
-                  const float* dt_bias, const float* a_log, const float* d_skip, const int* q_start,
-                  const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int G,
+                  const float* dt_bias, const float* a_log, const float* d_skip, const float* log_decay,
+                  const float* put, const int* q_start, const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int G,
                   int P, int N, cudaStream_t stream);
+int yalm_head_store(const float* qkv, int n_partials, long long partial_stride, const float* q_norm, const float* k_norm,
+                    float eps, int true_dk, const float* table, int dims, float temp_coef, float temp_every,
+                    const int* token_seq, const int* q_start, const int* seq_slot, const int* slot_pos, void* q_out,
+                    void* kv_step, void* k_cache, void* v_cache, int dtype, int n_tokens, int H, int G, int dk, int dv,
+                    int has_v, int capacity, int write_cache, const int* page_table, int pages_per_slot, int n_pages,
+                    cudaStream_t stream);
+int yalm_attention_kv(const void* q, const void* kv_step, const void* k_cache, const void* v_cache, const int* token_seq,
+                      const int* q_start, const int* seq_slot, const int* slot_pos, void* out, int dtype, int n_tokens,
+                      int n_seqs, int max_q_len, int H, int G, int dk, int dv, int capacity, float scale,
+                      const float* bias, int n_bias, const float* sink, int decode, int mma, int nsplit, float* part_o,
+                      float* part_ml, int* counters, int max_keys, int* status, const int* page_table,
+                      int pages_per_slot, int n_pages, cudaStream_t stream);
+int yalm_gla(const float* proj, int n_partials, long long partial_stride, int proj_row, int col_q, int col_k, int col_v,
+             int col_low, int rank, const float* w2, const float* bias, float inv_tau, float q_scale, float* act, int* marks,
+             const int* q_start, const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int dk,
+             int dv, cudaStream_t stream);
+int yalm_mlstm_prep(const float* proj, int n_partials, long long partial_stride, int proj_row, int col_q, int col_k,
+                    int col_v, int col_i, int col_f, const float* i_bias, const float* f_bias, float cap, float q_scale,
+                    float* act, float* log_decay, float* put, float* floor, float* maxima, const int* q_start,
+                    const int* seq_slot, int n_tokens, int n_seqs, int H, int dk, int dv, int P, cudaStream_t stream);
+int yalm_gated_heads(const float* y, const float* floor, const float* w, const float* gate, int gate_n,
+                     long long gate_stride, int gate_row, int col0, int silu, void* out, int out_dtype, int rows,
+                     int heads, int size, int pitch, float eps, cudaStream_t stream);
 int yalm_gated_group_norm(const float* y, const float* z, int z_n, long long z_stride, int z_row, int col0,
                           const float* w, void* out, int out_dtype, int rows, int inner, int groups,
                           float eps, cudaStream_t stream);
@@ -380,8 +403,8 @@ int yalm_activation_rows(const float* z, int n_partials, long long partial_strid
 
 
 // ---- norm_step.cu: sublayer outputs that are normed before they join the residual stream ------------
-int yalm_norm_step(float* x, const float* a, int na, long long sa, float fa, const float* b, int nb,
-                   long long sb, float fb, int post_kind, const float* post_w, const float* post_b,
+int yalm_norm_step(float* x, const float* a, int na, long long sa, float fa, const float* wa, const float* b, int nb,
+                   long long sb, float fb, const float* wb, const float* c, int nc, long long sc, float fc, const float* wc, int post_kind, const float* post_w, const float* post_b,
                    float post_alpha, float post_eps, int pre_kind, const float* pre_w, const float* pre_b,
                    float pre_alpha, float pre_eps, void* h, int h_dtype, const int* rows, int n_rows, int dim,
                    cudaStream_t stream);
@@ -396,9 +419,12 @@ int yalm_gated_rows(const float* z, int n_partials, long long partial_stride, co
 
 // ---- delta_rule.cu: the gated delta rule with a decay per key channel ------------------------------
 int yalm_delta_row(int H, int G, int dk, int dv);
-int yalm_delta_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row,
-                    int col_b, int col_low, int n_low, void* low, int low_dtype, int n_tokens, int H, int G,
-                    int dk, int dv, cudaStream_t stream);
+int yalm_delta_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row, int col_b,
+                    int col_low, int n_low, void* low, int low_dtype, int col_a, const float* dt_bias,
+                    const float* a_log, int n_tokens, int H, int G, int dk, int dv, cudaStream_t stream);
+int yalm_delta_head_row(int H, int G, int dk, int dv);
+int yalm_delta_head_scan(const float* act, const int* q_start, const int* seq_slot, float* state, float* out,
+                         int n_tokens, int n_seqs, int H, int G, int dk, int dv, cudaStream_t stream);
 int yalm_delta_scan(float* act, const float* z, int n_partials, long long partial_stride,
                     const float* dt_bias, const float* a_log, float* gate, const int* q_start,
                     const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int G,

@@ -2,7 +2,9 @@
 // (x <- x + post(y)) and norm the stream again for the next sublayer (h = pre(x)):
 //
 //  * norm_step: one pass over a row does the write that is due and the read that follows,
-//        y = f_A sum(slices A) + f_B sum(slices B)          (a mixer of two branches hands two sets)
+//        y = f_A w_A sum(slices A) + f_B w_B sum(slices B) + f_C w_C sum(slices C)
+//                         (up to three sets: a mixer of two branches hands two, a feed-forward beside it the
+//                         third; w, a factor per feature, may be absent)
 //        x <- x + post(y),   h = pre(x)
 //    where post and pre are each one of
 //        tanh form ("dynamic tanh"):  n(v) = tanh(alpha v) w + b       no mean, no variance
@@ -35,6 +37,10 @@ struct SliceSet {
   int n;
   long long stride;
   float factor;
+  const float* w;        // a factor per feature, or null
+};
+struct SliceSets {
+  SliceSet s[3];
 };
 
 __device__ __forceinline__ float apply_tanh_form(const NormForm& f, float v, int i) {
@@ -53,6 +59,34 @@ __device__ __forceinline__ float4 slices4(const float* __restrict__ p, int n, lo
     for (int j = 0; j < 4; ++j) { v.x += t[j].x; v.y += t[j].y; v.z += t[j].z; v.w += t[j].w; }
   }
   return v;
+}
+// y at four neighbouring features (or one) of row t
+__device__ __forceinline__ float4 sets4(const SliceSets& sets, size_t at, int i) {
+  float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {
+    const SliceSet& a = sets.s[k];
+    if (a.p == nullptr) continue;
+    const float4 v = slices4(a.p + at, a.n, a.stride);
+    float4 f = make_float4(a.factor, a.factor, a.factor, a.factor);
+    if (a.w != nullptr) {
+      const float4 w = *reinterpret_cast<const float4*>(a.w + i);
+      f.x *= w.x; f.y *= w.y; f.z *= w.z; f.w *= w.w;
+    }
+    y.x = fmaf(f.x, v.x, y.x); y.y = fmaf(f.y, v.y, y.y); y.z = fmaf(f.z, v.z, y.z); y.w = fmaf(f.w, v.w, y.w);
+  }
+  return y;
+}
+__device__ __forceinline__ float sets1(const SliceSets& sets, size_t at, int i) {
+  float y = 0.f;
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {
+    const SliceSet& a = sets.s[k];
+    if (a.p == nullptr) continue;
+    const float f = a.w != nullptr ? a.factor * a.w[i] : a.factor;
+    y = fmaf(f, sum_slices(a.p + at, a.n, a.stride), y);
+  }
+  return y;
 }
 template <typename T>
 __device__ __forceinline__ void store4(T* __restrict__ p, float a, float b, float c, float d) {
@@ -81,7 +115,7 @@ __device__ __forceinline__ float row_deviations(const float* row, float mean, in
 
 // VEC: dim is a multiple of four and every pointer 16-byte aligned: a thread takes four neighbouring features
 template <typename T, bool VEC>
-__global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, NormForm post, NormForm pre,
+__global__ void norm_step_kernel(float* __restrict__ x, SliceSets sets, NormForm post, NormForm pre,
                                  T* __restrict__ h, const int* __restrict__ rows, int dim) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float row_s[];           // the row: y, then the new x
@@ -97,15 +131,10 @@ __global__ void norm_step_kernel(float* __restrict__ x, SliceSet A, SliceSet B, 
     for (int i = i0; i < dim; i += step) {
       float y[W];
       if constexpr (VEC) {
-        float4 ya = make_float4(0.f, 0.f, 0.f, 0.f), yb = ya;
-        if (A.p != nullptr) ya = slices4(A.p + t * dim + i, A.n, A.stride);
-        if (B.p != nullptr) yb = slices4(B.p + t * dim + i, B.n, B.stride);
-        y[0] = fmaf(B.factor, yb.x, A.factor * ya.x); y[1] = fmaf(B.factor, yb.y, A.factor * ya.y);
-        y[2] = fmaf(B.factor, yb.z, A.factor * ya.z); y[3] = fmaf(B.factor, yb.w, A.factor * ya.w);
+        const float4 v = sets4(sets, t * dim + i, i);
+        y[0] = v.x; y[1] = v.y; y[2] = v.z; y[3] = v.w;
       } else {
-        y[0] = 0.f;
-        if (A.p != nullptr) y[0] = A.factor * sum_slices(A.p + t * dim + i, A.n, A.stride);
-        if (B.p != nullptr) y[0] = fmaf(B.factor, sum_slices(B.p + t * dim + i, B.n, B.stride), y[0]);
+        y[0] = sets1(sets, t * dim + i, i);
       }
 #pragma unroll
       for (int j = 0; j < W; ++j) { row_s[i + j] = y[j]; ss += post.kind == 4 ? y[j] : y[j] * y[j]; }
@@ -186,7 +215,7 @@ __device__ __forceinline__ float row_sum(float v, float* part) {
 }
 
 template <typename T, int E>
-__global__ void norm_step_reg_kernel(float* __restrict__ x, SliceSet A, SliceSet B, NormForm post, NormForm pre,
+__global__ void norm_step_reg_kernel(float* __restrict__ x, SliceSets sets, NormForm post, NormForm pre,
                                      T* __restrict__ h, const int* __restrict__ rows, int dim) {
   pdl_launch_dependents();
   __shared__ float parts[4][32];
@@ -206,13 +235,8 @@ __global__ void norm_step_reg_kernel(float* __restrict__ x, SliceSet A, SliceSet
 #pragma unroll
     for (int e = 0; e < E; ++e) {
       const int i = (threadIdx.x + e * blockDim.x) * 4;
-      float4 ya = make_float4(0.f, 0.f, 0.f, 0.f), yb = ya;
-      if (i < dim) {
-        if (A.p != nullptr) ya = slices4(A.p + t * dim + i, A.n, A.stride);
-        if (B.p != nullptr) yb = slices4(B.p + t * dim + i, B.n, B.stride);
-      }
-      y[e][0] = fmaf(B.factor, yb.x, A.factor * ya.x); y[e][1] = fmaf(B.factor, yb.y, A.factor * ya.y);
-      y[e][2] = fmaf(B.factor, yb.z, A.factor * ya.z); y[e][3] = fmaf(B.factor, yb.w, A.factor * ya.w);
+      const float4 v4 = i < dim ? sets4(sets, t * dim + i, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      y[e][0] = v4.x; y[e][1] = v4.y; y[e][2] = v4.z; y[e][3] = v4.w;
 #pragma unroll
       for (int j = 0; j < 4; ++j) s1 += post.kind == 4 ? y[e][j] : y[e][j] * y[e][j];
     }
@@ -483,24 +507,26 @@ __global__ void gated_rows_kernel(const float* __restrict__ z, int n_partials, l
 
 using namespace yalm;
 
-// x float32 [.., dim] (changed in place when post_kind != 0).  y = fa * sum(slices a) + fb * sum(slices b)
-// (either may be null).  post / pre: kind 0 absent, 1 tanh form (w, b, alpha), 2 rms form (w, eps),
+// x float32 [.., dim] (changed in place when post_kind != 0).  y = sum over a, b, c of f * w * sum(slices)
+// (any may be null; w float32 [dim] or null).  post / pre: kind 0 absent, 1 tanh form (w, b, alpha), 2 rms form (w, eps),
 // 3 none, 4 layer form (w, eps).  h [n_rows][dim] in h_dtype receives pre(x).  rows (optional, only without a post step): the
 // rows of x that are read.
-extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, float fa, const float* b,
-                              int nb, long long sb, float fb, int post_kind, const float* post_w,
+extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, float fa, const float* wa,
+                              const float* b, int nb, long long sb, float fb, const float* wb, const float* c,
+                              int nc, long long sc, float fc, const float* wc, int post_kind, const float* post_w,
                               const float* post_b, float post_alpha, float post_eps, int pre_kind,
                               const float* pre_w, const float* pre_b, float pre_alpha, float pre_eps,
                               void* h, int h_dtype, const int* rows, int n_rows, int dim,
                               cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (dim <= 0 || dim > 12288 || (rows != nullptr && post_kind) || (!post_kind && !pre_kind)) return -2;
-  if ((post_kind && a == nullptr && b == nullptr) || (pre_kind && h == nullptr)) return -2;
-  const SliceSet A = {a, na, sa, fa}, B = {b, nb, sb, fb};
+  if ((post_kind && a == nullptr && b == nullptr && c == nullptr) || (pre_kind && h == nullptr)) return -2;
+  const SliceSets sets = {{{a, na, sa, fa, wa}, {b, nb, sb, fb, wb}, {c, nc, sc, fc, wc}}};
   const NormForm post = {post_kind, post_w, post_b, post_alpha, post_eps};
   const NormForm pre = {pre_kind, pre_w, pre_b, pre_alpha, pre_eps};
-  const bool vec = dim % 4 == 0 && (sa & 3) == 0 && (sb & 3) == 0 &&
-                   ((((uintptr_t)x) | ((uintptr_t)a) | ((uintptr_t)b) | ((uintptr_t)h)) & 15) == 0;
+  const bool vec = dim % 4 == 0 && (sa & 3) == 0 && (sb & 3) == 0 && (sc & 3) == 0 &&
+                   ((((uintptr_t)x) | ((uintptr_t)a) | ((uintptr_t)b) | ((uintptr_t)c) | ((uintptr_t)h) | ((uintptr_t)wa) |
+                     ((uintptr_t)wb) | ((uintptr_t)wc)) & 15) == 0;
   const dim3 grid(n_rows);
   if (vec && dim <= 8192 && ((((uintptr_t)post_w) | ((uintptr_t)pre_w)) & 15) == 0) {
     // many rows: four groups of four features per thread, so that many rows are in flight on an SM; few: one
@@ -509,9 +535,9 @@ extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, fl
     const dim3 block(((groups + e - 1) / e + 31) / 32 * 32);
 #define YALM_NSR(T)                                                                                            \
   do {                                                                                                         \
-    if (e == 4) launch_pdl(norm_step_reg_kernel<T, 4>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim); \
-    else if (e == 2) launch_pdl(norm_step_reg_kernel<T, 2>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim); \
-    else launch_pdl(norm_step_reg_kernel<T, 1>, grid, block, 0, stream, x, A, B, post, pre, (T*)h, rows, dim);  \
+    if (e == 4) launch_pdl(norm_step_reg_kernel<T, 4>, grid, block, 0, stream, x, sets, post, pre, (T*)h, rows, dim); \
+    else if (e == 2) launch_pdl(norm_step_reg_kernel<T, 2>, grid, block, 0, stream, x, sets, post, pre, (T*)h, rows, dim); \
+    else launch_pdl(norm_step_reg_kernel<T, 1>, grid, block, 0, stream, x, sets, post, pre, (T*)h, rows, dim);  \
   } while (0)
     if (h_dtype == DT_F32) YALM_NSR(float);
     else if (h_dtype == DT_BF16) YALM_NSR(__nv_bfloat16);
@@ -535,7 +561,7 @@ extern "C" int yalm_norm_step(float* x, const float* a, int na, long long sa, fl
       if (e != cudaSuccess) return (int)e;                                                            \
       attr = smem;                                                                                    \
     }                                                                                                 \
-    launch_pdl(norm_step_kernel<T, V>, grid, block, smem, stream, x, A, B, post, pre, (T*)h, rows, dim); \
+    launch_pdl(norm_step_kernel<T, V>, grid, block, smem, stream, x, sets, post, pre, (T*)h, rows, dim); \
   } while (0)
 #define YALM_NS(T)                \
   do {                            \

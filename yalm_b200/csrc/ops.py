@@ -127,16 +127,23 @@ _SIGNATURES = {
     "yalm_latent_prefill_usable": [_i, _i, _i, _i, _i, _i],
     "yalm_latent_prefill": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _i, _i, _ll,
                             _i, _i, _vp],
-    "yalm_ssd_scan": [_vp, _vp, _i, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "yalm_ssd_scan": [_vp, _vp, _i, _ll, _i, _i] + [_vp] * 9 + [_i] * 6 + [_vp],
+    "yalm_gla": [_vp, _i, _ll, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _f] + [_vp] * 6 + [_i] * 5 + [_vp],
+    "yalm_mlstm_prep": [_vp, _i, _ll, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _f] + [_vp] * 7 + [_i] * 6 + [_vp],
+    "yalm_gated_heads": [_vp, _vp, _vp, _vp, _i, _ll, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp],
+    "yalm_head_store": [_vp, _i, _ll, _vp, _vp, _f, _i, _vp, _i, _f, _f] + [_vp] * 8 + [_i] * 9 + [_vp, _i, _i, _vp],
+    "yalm_attention_kv": [_vp] * 9 + [_i] * 9 + [_f, _vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _vp],
+    "yalm_delta_head_row": [_i, _i, _i, _i],
+    "yalm_delta_head_scan": [_vp] * 5 + [_i] * 6 + [_vp],
     "yalm_gated_group_norm": [_vp, _vp, _i, _ll, _i, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "yalm_activation_rows": [_vp, _i, _ll, _vp, _i, _ll, _i, _vp],
-    "yalm_norm_step": [_vp, _vp, _i, _ll, _f, _vp, _i, _ll, _f, _i, _vp, _vp, _f, _f, _i, _vp, _vp, _f, _f, _vp,
+    "yalm_norm_step": [_vp] + [_vp, _i, _ll, _f, _vp] * 3 + [_i, _vp, _vp, _f, _f, _i, _vp, _vp, _f, _f, _vp,
                        _i, _vp, _i, _i, _vp],
     "yalm_short_conv": [_vp, _i, _ll, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _vp,
                         _i, _i, _i, _i, _i, _vp],
     "yalm_gated_rows": [_vp, _i, _ll, _vp, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp],
     "yalm_delta_row": [_i, _i, _i, _i],
-    "yalm_delta_prep": [_vp, _vp, _i, _ll, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "yalm_delta_prep": [_vp, _vp, _i, _ll, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "yalm_delta_scan": [_vp, _vp, _i, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "yalm_rglru": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _ll, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
                    _f, _vp],
@@ -1125,23 +1132,178 @@ def latent_prefill(q: torch.Tensor, kv: torch.Tensor, kv_step: torch.Tensor, bat
 
 
 # ---- a state-space recurrence with one decay per head ------------------------------------------------
-def ssd_scan(act: torch.Tensor, dt: torch.Tensor, n_partials: int, col0: int, dt_bias: torch.Tensor,
-             a_log: torch.Tensor, d_skip: torch.Tensor, batch, state: torch.Tensor, out: torch.Tensor, H: int, G: int,
-             P: int, N: int) -> None:
+def ssd_scan(act: torch.Tensor, dt: Optional[torch.Tensor], n_partials: int, col0: int, dt_bias: Optional[torch.Tensor],
+             a_log: Optional[torch.Tensor], d_skip: Optional[torch.Tensor], batch, state: torch.Tensor,
+             out: torch.Tensor, H: int, G: int, P: int, N: int, steps=None) -> None:
     """S_t = exp(-exp(a_log) dt_t) S_(t-1) + dt_t B_t x_t^T, out_t = S_t^T C_t + d_skip x_t per head (head h with
     group h // (H / G)) over the step's tokens.  act float32 [N, H P + 2 G N] = (x | B | C); dt = softplus(column
     col0 + h of the slices ``dt`` float32 [(s,) N, row] + dt_bias); ``state`` float32 [slots, H, P, N] is read at
-    the step's start and written at its end; out float32 [N, H P]."""
+    the step's start and written at its end; out float32 [N, H P].  ``steps`` = (logarithms of the decays, at most
+    0 but for rounding; factors in place of dt_t), both float32 [N, H], instead of ``dt``, ``dt_bias`` and
+    ``a_log`` (None).  ``d_skip`` may be None."""
     n = batch.n_tokens
     _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, H * P + 2 * G * N)
           and out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, H * P)
           and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, P, N),
           "ssd_scan: shapes")
-    for v in (dt_bias, a_log, d_skip):
-        _need(v.dtype == torch.float32 and v.numel() == H and v.is_contiguous(), "ssd_scan: float32 [H]")
-    src, s, stride, row, c = _columns(dt, n_partials, n, col0, H, "ssd_scan: step columns")
-    _check(lib().yalm_ssd_scan(_p(act), src, s, stride, row, c, _p(dt_bias), _p(a_log), _p(d_skip), _p(batch.q_start),
+    for v in (d_skip,) if steps is not None else (dt_bias, a_log, d_skip):
+        _need(v is None or (v.dtype == torch.float32 and v.numel() == H and v.is_contiguous()), "ssd_scan: float32 [H]")
+    if steps is None:
+        src = _columns(dt, n_partials, n, col0, H, "ssd_scan: step columns")
+        la = put = None
+    else:
+        src = (None, 0, 0, 0, 0)
+        la, put = steps
+        for v in steps:
+            _need(v.dtype == torch.float32 and v.is_contiguous() and tuple(v.shape) == (n, H), "ssd_scan: steps [N, H]")
+    _check(lib().yalm_ssd_scan(_p(act), *src, _p(dt_bias), _p(a_log), _p(d_skip), _p(la), _p(put), _p(batch.q_start),
                                _p(batch.seq_slot), _p(state), _p(out), n, batch.n_seqs, H, G, P, N, _stream()), "ssd_scan")
+
+
+def gla(proj: torch.Tensor, n_partials: int, cols, rank: int, w2: torch.Tensor, bias: torch.Tensor, tau: float,
+        act: torch.Tensor, marks: torch.Tensor, batch, state: torch.Tensor, out: torch.Tensor, H: int, dk: int,
+        dv: int) -> None:
+    """Gated linear attention over the step's tokens: S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, out_t = S_t^T q_t
+    dk^-1/2 per head, log alpha = logsigmoid(W2 low + bias) / tau.  proj: float32 slices [(s,) N, row] with q, k,
+    v and low at the columns ``cols``; w2 float32 [rank, H dk]; act float32 [N, 3 H dk + H dv] and marks int32
+    [N, H] are scratch; state float32 [slots, H, dv, dk] is read at the step's start and written at its end;
+    out float32 [N, H dv]."""
+    n, row = batch.n_tokens, proj.shape[-1]
+    cq, ck, cv, cl = (int(c) for c in cols)
+    _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[-2] == n
+          and max(cq + H * dk, ck + H * dk, cv + H * dv, cl + rank) <= row, "gla: columns of proj")
+    _need(w2.dtype == bias.dtype == torch.float32 and w2.is_contiguous() and tuple(w2.shape) == (rank, H * dk)
+          and bias.numel() == H * dk, "gla: w2 [rank, H dk], bias [H dk]")
+    _need(act.dtype == torch.float32 and act.is_contiguous() and act.numel() >= n * (3 * H * dk + H * dv)
+          and marks.dtype == torch.int32 and marks.numel() >= n * H, "gla: scratch")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
+          and out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, H * dv), "gla: state, out")
+    _check(lib().yalm_gla(_p(proj), int(n_partials), n * row, row, cq, ck, cv, cl, rank, _p(w2), _p(bias), 1.0 / float(tau),
+                          float(dk) ** -0.5, _p(act), _p(marks), _p(batch.q_start), _p(batch.seq_slot), _p(state), _p(out),
+                          n, batch.n_seqs, H, dk, dv, _stream()), "gla", kernels=2)
+
+
+def mlstm_prep(proj: torch.Tensor, n_partials: int, cols, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+               act: torch.Tensor, log_decay: torch.Tensor, put: torch.Tensor, floor: torch.Tensor, maxima: torch.Tensor,
+               batch, H: int, dk: int, dv: int, P: int) -> None:
+    """The matrix memory's gates and rows for ``ssd_scan``: m_t = max(f_t + m_(t-1), i_t) with i = cap tanh((z_i +
+    i_bias) / cap) and f = logsigmoid(cap tanh((z_f + f_bias) / cap)); log_decay = f_t + m_(t-1) - m_t, put = exp(i_t
+    - m_t), floor = exp(-m_t), float32 [N, H]; act float32 [N, H P + 2 H dk] = (v, 1, 0 .. | k | q dk^-1/2).  proj:
+    float32 slices with q, k, v, i, f at the columns ``cols``; maxima float32 [slots, H] is read at the step's
+    start and written at its end."""
+    n, row = batch.n_tokens, proj.shape[-1]
+    cq, ck, cv, ci, cf = (int(c) for c in cols)
+    _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[-2] == n
+          and max(cq + H * dk, ck + H * dk, cv + H * dv, ci + H, cf + H) <= row, "mlstm_prep: columns of proj")
+    for v in (i_bias, f_bias):
+        _need(v.dtype == torch.float32 and v.numel() == H, "mlstm_prep: biases float32 [H]")
+    for v in (log_decay, put, floor):
+        _need(v.dtype == torch.float32 and v.is_contiguous() and tuple(v.shape) == (n, H), "mlstm_prep: [N, H]")
+    _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, H * P + 2 * H * dk) and P > dv
+          and maxima.dtype == torch.float32 and maxima.is_contiguous() and tuple(maxima.shape[1:]) == (H,),
+          "mlstm_prep: act, maxima")
+    _check(lib().yalm_mlstm_prep(_p(proj), int(n_partials), n * row, row, cq, ck, cv, ci, cf, _p(i_bias), _p(f_bias),
+                                 float(cap), float(dk) ** -0.5, _p(act), _p(log_decay), _p(put), _p(floor), _p(maxima),
+                                 _p(batch.q_start), _p(batch.seq_slot), n, batch.n_seqs, H, dk, dv, P, _stream()),
+           "mlstm_prep")
+
+
+def gated_heads(y: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, n_partials: int, col0: int,
+                out: torch.Tensor, heads: int, size: int, eps: float, silu: bool,
+                floor: Optional[torch.Tensor] = None) -> None:
+    """out [N, heads size] = every head's ``size`` values of y over their root mean square, times weight [heads
+    size], times the sigmoid (or SiLU) of the ``heads size`` columns from col0 of float32 slices ``gate``.  y
+    float32 [N, heads pitch]; with ``floor`` [N, heads] a head's values are first divided by max(|the value after
+    them|, floor) + 1e-6."""
+    n = y.shape[0]
+    pitch = y.shape[1] // heads
+    _need(y.dtype == weight.dtype == torch.float32 and y.is_contiguous() and y.shape[1] == heads * pitch
+          and pitch >= size + (floor is not None) and weight.numel() == heads * size and weight.is_contiguous()
+          and out.is_contiguous() and tuple(out.shape) == (n, heads * size), "gated_heads: shapes")
+    _need(floor is None or (floor.dtype == torch.float32 and floor.is_contiguous() and tuple(floor.shape) == (n, heads)),
+          "gated_heads: floor")
+    src, s, stride, row, c = _columns(gate, n_partials, n, col0, heads * size, "gated_heads: gate columns")
+    _check(lib().yalm_gated_heads(_p(y), _p(floor), _p(weight), src, s, stride, row, c, int(silu), _p(out),
+                                  dtype_code(out.dtype), n, heads, size, pitch, float(eps), _stream()), "gated_heads")
+
+
+def head_store(qkv: torch.Tensor, n_partials: int, norms, table: Optional[torch.Tensor], dims: int, temperature, batch,
+               slot_pos: torch.Tensor, q_out: torch.Tensor, kv_step: torch.Tensor, k_cache: torch.Tensor,
+               v_cache: torch.Tensor, H: int, G: int, dk: int, dv: int, has_v: bool, capacity: int,
+               pages: Optional[torch.Tensor] = None) -> None:
+    """Sums the slices of a q/k(/v) product float32 [(s,) N, H dk + G dk (+ G dv)], norms each head of q and k with
+    ``norms`` = (q weight [dk], k weight [dk], eps, true size) or None, turns the first ``dims`` features in halves
+    by ``table`` float32 [N, dims / 2, 2], multiplies q by 1 + coef ln(floor((pos + 1) / every) + 1) with
+    ``temperature`` = (coef, every) or None, and writes q_out [N, H, dk], kv_step [N, G dk + G dv] and the caches
+    ([.., dk] and [.., dv] rows).  Without v columns a value is its key as projected."""
+    n = batch.n_tokens
+    row = H * dk + G * dk + (G * dv if has_v else 0)
+    _need(qkv.dtype == torch.float32 and qkv.is_contiguous() and qkv.numel() >= n_partials * n * row, "head_store: slices")
+    _need(q_out.dtype == kv_step.dtype == k_cache.dtype == v_cache.dtype and q_out.is_contiguous()
+          and q_out.numel() == n * H * dk and kv_step.is_contiguous() and kv_step.numel() == n * G * (dk + dv),
+          "head_store: outputs")
+    _need(k_cache.shape[-1] == dk and v_cache.shape[-1] == dv, "head_store: cache rows")
+    qn, kn, eps, true_dk = norms if norms is not None else (None, None, 0.0, dk)
+    for v in (qn, kn):
+        _need(v is None or (v.dtype == torch.float32 and v.numel() == dk), "head_store: norm weights float32 [dk]")
+    _need(not dims or (table is not None and table.dtype == torch.float32 and table.numel() == n * dims), "head_store: table")
+    coef, every = temperature if temperature is not None else (0.0, 0.0)
+    pt, pps, n_pages = _pages(pages, k_cache, G, dk)
+    _check(lib().yalm_head_store(_p(qkv), int(n_partials), n * row, _p(qn), _p(kn), float(eps), int(true_dk), _p(table),
+                                 int(dims), float(coef), float(every), _p(batch.token_seq), _p(batch.q_start),
+                                 _p(batch.seq_slot), _p(slot_pos), _p(q_out), _p(kv_step), _p(k_cache), _p(v_cache),
+                                 dtype_code(q_out.dtype), n, H, G, dk, dv, int(has_v), int(capacity), 1, pt, pps, n_pages,
+                                 _stream()), "head_store")
+
+
+def attention_kv(q: torch.Tensor, kv_step: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, batch,
+                 slot_pos: torch.Tensor, out: torch.Tensor, H: int, G: int, dk: int, dv: int, capacity: int,
+                 scale: float, status: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                 sink: Optional[torch.Tensor] = None, mma: bool = True, nsplit: int = 1,
+                 part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
+                 counters: Optional[torch.Tensor] = None, max_keys: int = 1 << 30,
+                 pages: Optional[torch.Tensor] = None) -> None:
+    """Causal attention with 32-bit scores, weights and sums, key size dk and value size dv: q [N, H, dk], kv_step
+    [N, G dk + G dv], out [N, H, dv].  score = scale q.k (+ bias[h][min(distance, last)], bias float32 [H, n]);
+    ``sink`` float32 [H] joins the denominator.  ``mma`` False: the FMA kernel.  ``nsplit`` > 1 (a decode step, or
+    the FMA kernel): a query's keys over so many blocks, with scratch part_o [N, H, nsplit, dv], part_ml [N, H,
+    nsplit, 2] and zeroed counters."""
+    n = batch.n_tokens
+    _need(q.dtype == kv_step.dtype == k_cache.dtype == v_cache.dtype == out.dtype and q.numel() == n * H * dk
+          and out.is_contiguous() and out.numel() == n * H * dv and kv_step.numel() == n * G * (dk + dv)
+          and k_cache.shape[-1] == dk and v_cache.shape[-1] == dv, "attention_kv: shapes")
+    n_bias = 0
+    if bias is not None:
+        n_bias = bias.shape[1]
+        _need(bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[0] == H, "attention_kv: bias [H, n]")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == H), "attention_kv: sink [H]")
+    if nsplit > 1:
+        _need(part_o.numel() >= n * H * nsplit * dv and part_ml.numel() >= 2 * n * H * nsplit
+              and counters.numel() >= n * G * -(-(H // G) // 4), "attention_kv: scratch")
+    pt, pps, n_pages = _pages(pages, k_cache, G, dk)
+    _check(lib().yalm_attention_kv(_p(q), _p(kv_step), _p(k_cache), _p(v_cache), _p(batch.token_seq), _p(batch.q_start),
+                                   _p(batch.seq_slot), _p(slot_pos), _p(out), dtype_code(q.dtype), n, batch.n_seqs,
+                                   max(batch.q_lens), H, G, dk, dv, int(capacity), float(scale), _p(bias), n_bias,
+                                   _p(sink), int(batch.is_decode), int(mma), int(nsplit), _p(part_o), _p(part_ml),
+                                   _p(counters), int(max_keys), _p(status), pt, pps, n_pages, _stream()), "attention_kv")
+
+
+def delta_head_row(H: int, G: int, dk: int, dv: int) -> int:
+    """Floats of a token's row for ``delta_head_scan``."""
+    return int(lib().yalm_delta_head_row(H, G, dk, dv))
+
+
+def delta_head_scan(act: torch.Tensor, batch, state: torch.Tensor, out: torch.Tensor, H: int, G: int, dk: int,
+                    dv: int) -> None:
+    """The gated delta rule with one decay per head over the step's tokens: act float32 [N, delta_head_row] = (q |
+    k | v | beta | log decay), state float32 [slots, H, dv, dk], out float32 [N, H dv]."""
+    n = batch.n_tokens
+    _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, delta_head_row(H, G, dk, dv))
+          and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
+          and out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (n, H * dv),
+          "delta_head_scan: shapes")
+    _check(lib().yalm_delta_head_scan(_p(act), _p(batch.q_start), _p(batch.seq_slot), _p(state), _p(out), n, batch.n_seqs,
+                                      H, G, dk, dv, _stream()), "delta_head_scan")
 
 
 def gated_group_norm(y: torch.Tensor, z: torch.Tensor, n_partials: int, col0: int, weight: torch.Tensor,
@@ -1176,21 +1338,25 @@ def norm_step(x: torch.Tensor, sets=(), post: Optional[tuple] = None, pre: Optio
               h: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
               n_rows: Optional[int] = None) -> None:
     """One pass over the rows of x float32 [N, dim]: x <- x + post(y), then h = pre(x).  y is the sum
-    over ``sets`` (up to two (slices float32 [S, N, dim], S, factor)) of factor * sum of slices.  ``post``
+    over ``sets`` (up to three (slices float32 [S, N, dim], S, factor), or with a factor per feature float32 [dim]
+    as a fourth member) of factor * sum of slices.  ``post``
     and ``pre`` are (kind, weight, bias, alpha, eps) with kind NORM_TANH (tanh(alpha v) w + b),
     NORM_RMS (v / sqrt(mean v^2 + eps) w), NORM_LAYER ((v - mean) / sqrt(mean (v - mean)^2 + eps) w) or
     NORM_NONE, or None for a step without that half.  With
     ``rows`` (int32 row numbers; no post half) only those rows are read: h [n_rows, dim]."""
     n, dim = x.shape
     _need(x.dtype == torch.float32 and x.is_contiguous(), "norm_step: x float32 [N, dim]")
-    _need(len(sets) <= 2 and (post is None) == (len(sets) == 0), "norm_step: a post step has one or two sets")
+    _need(len(sets) <= 3 and (post is None) == (len(sets) == 0), "norm_step: a post step has one to three sets")
     args = []
-    for buf, S, factor in sets:
+    for buf, S, factor, *rest in sets:
+        w = rest[0] if rest else None
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == dim),
+              "norm_step: a set's weight is float32 [dim]")
         _need(buf.dtype == torch.float32 and buf.is_contiguous() and buf.numel() >= S * n * dim,
               "norm_step: a set is float32 [S, N, dim]")
-        args += [_p(buf), int(S), n * dim, float(factor)]
-    while len(args) < 8:
-        args += [None, 0, 0, 0.0]
+        args += [_p(buf), int(S), n * dim, float(factor), _p(w)]
+    while len(args) < 15:
+        args += [None, 0, 0, 0.0, None]
     forms = []
     for f in (post, pre):
         if f is None:
@@ -1264,19 +1430,24 @@ def delta_row(H: int, G: int, dk: int, dv: int) -> int:
 
 
 def delta_prep(act: torch.Tensor, proj: torch.Tensor, n_partials: int, col_b: int, col_low: int, n_low: int,
-               low: torch.Tensor, H: int, G: int, dk: int, dv: int) -> None:
+               low: Optional[torch.Tensor], H: int, G: int, dk: int, dv: int, head_decay=None) -> None:
     """act float32 [N, delta_row] holds q | k | v (after convolution and SiLU) in its first columns: q and
     k become unit vectors per head (q also times dk^-1/2), beta = sigmoid of the H columns of ``proj``
     (float32 slices [(s,) N, row]) from col_b, and the n_low columns from col_low go to ``low`` [N, n_low]
-    in low's type."""
+    in low's type.  ``head_decay`` = (column of the H decay logits, dt_bias [H], a_log [H]): the rows are
+    those of ``delta_head_scan`` and receive the logarithms of the decays."""
     n = act.shape[0]
-    _need(act.dtype == torch.float32 and act.is_contiguous() and act.shape[1] == delta_row(H, G, dk, dv)
+    want = delta_row(H, G, dk, dv) if head_decay is None else delta_head_row(H, G, dk, dv)
+    _need(act.dtype == torch.float32 and act.is_contiguous() and act.shape[1] == want
           and proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[-2] == n
-          and low.is_contiguous() and tuple(low.shape) == (n, n_low), "delta_prep: shapes")
+          and (n_low == 0 or (low.is_contiguous() and tuple(low.shape) == (n, n_low))), "delta_prep: shapes")
+    col_a, dt_bias, a_log = head_decay if head_decay is not None else (0, None, None)
+    for v in (dt_bias, a_log):
+        _need(v is None or (v.dtype == torch.float32 and v.numel() == H), "delta_prep: dt_bias, a_log float32 [H]")
     row = proj.shape[-1]
     _check(lib().yalm_delta_prep(_p(act), _p(proj), int(n_partials), n * row, row, int(col_b), int(col_low),
-                                 int(n_low), _p(low), dtype_code(low.dtype), n, H, G, dk, dv, _stream()),
-           "delta_prep")
+                                 int(n_low), _p(low), dtype_code(low.dtype) if low is not None else F32, int(col_a),
+                                 _p(dt_bias), _p(a_log), n, H, G, dk, dv, _stream()), "delta_prep")
 
 
 def delta_scan(act: torch.Tensor, z: torch.Tensor, n_partials: int, dt_bias: torch.Tensor, a_log: torch.Tensor,

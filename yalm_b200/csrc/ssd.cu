@@ -23,53 +23,24 @@
 //
 // The state is kept as [slots][H][P][N]: a column's rows are neighbours, which is how lanes own them.
 #include "api.h"
-#include "common.cuh"
+#include "scan.cuh"
 
 namespace yalm {
 
-constexpr int SS_TOK = 16, SS_STAGES = 3, SS_RUN = 8, SS_CPL = 4, SS_COLS = 8 * SS_CPL;
 constexpr float SS_SPAN = 16.f;
-
-typedef unsigned long long f2;                           // two packed floats
-__device__ __forceinline__ f2 pack_f2(float lo, float hi) {
-  f2 r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-  return r;
-}
-__device__ __forceinline__ void unpack_f2(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
-__device__ __forceinline__ f2 fma_f2(f2 a, f2 b, f2 c) {
-  f2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ f2 mul_f2(f2 a, f2 b) {
-  f2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-template <int BYTES>
-__device__ __forceinline__ void ss_copy(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(smem_u32(dst)), "l"(src), "n"(BYTES) : "memory");
-}
 
 struct SsdArgs {
   const float* act;            // [tokens][H P + 2 G N] = (x | B | C), after the convolution
   const float* dt;             // slices [dt_n][tokens][dt_row], one raw step per head
   int dt_n, dt_row;
   long long dt_stride;
-  const float *dt_bias, *a_log, *d_skip;       // [H]
+  const float *dt_bias, *a_log, *d_skip;       // [H]; d_skip may be null
+  const float *log_decay, *put;                // [tokens][H]: a_t and dt_t as they are, in place of the four above
   const int *q_start, *seq_slot;
   float* state;                // [slots][H][P][N]
   float* out;                  // [tokens][H P]
   int H, G, P, N;
 };
-
-__device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-
-// A decay exp(a), a <= 0, as it is applied: S <- coef S + keep S, with keep 1 where coef = exp(a) - 1 (its sign
-// bit is set, also for a = -0) and 0 where coef = exp(a)
-__device__ __forceinline__ float decay_coef(float a) { return a > -0.69f ? expm1f(a) : expf(a); }
-__device__ __forceinline__ float decay_keep(float coef) { return signbit(coef) ? 1.f : 0.f; }
 
 // K4: groups of four rows per lane (64 K4 >= N); VEC: N, P and the pointers allow 16-byte accesses
 template <int K4, bool VEC>
@@ -96,7 +67,8 @@ ssd_scan_kernel(SsdArgs a) {
   const int n_groups = (t1 - t0 + SS_TOK - 1) / SS_TOK;
   if (warp == 4) {                                       // the warp that feeds the others
     const int row = inner + 2 * a.G * N, g = h / (a.H / a.G);
-    const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h];
+    const bool given = a.put != nullptr;
+    const float neg_a = given ? 0.f : -expf(a.a_log[h]), bias = given ? 0.f : a.dt_bias[h];
     constexpr int W = VEC ? 4 : 1;
     const int per = (2 * N + min(SS_COLS, P - c0)) / W;  // copies per token
     auto issue = [&](int gi) {
@@ -118,11 +90,13 @@ ssd_scan_kernel(SsdArgs a) {
     };
     auto load_dt = [&](int gi) {
       const int t = t0 + gi * SS_TOK + lane;
-      return (lane < SS_TOK && t < t1) ? sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) : 0.f;
+      if (lane >= SS_TOK || t >= t1) return make_float2(0.f, -0.f);
+      if (given) return make_float2(a.put[(size_t)t * a.H + h], a.log_decay[(size_t)t * a.H + h]);
+      return make_float2(sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride), 0.f);
     };
-    auto put_dt = [&](int gi, float raw) {
-      const float dt = softplus(raw + bias);
-      const float la = neg_a * dt;
+    auto put_dt = [&](int gi, float2 raw) {
+      const float dt = given ? raw.x : softplus(raw.x + bias);
+      const float la = given ? raw.y : neg_a * dt;
       float cum = la;                                    // the run's inclusive sum
 #pragma unroll
       for (int o = 1; o < SS_RUN; o <<= 1) {
@@ -135,12 +109,12 @@ ssd_scan_kernel(SsdArgs a) {
         if ((lane & (SS_RUN - 1)) == SS_RUN - 1) run_s[gi % SS_STAGES][lane / SS_RUN] = make_float2(cum, decay_coef(cum));
       }
     };
-    float raw0 = load_dt(0), raw1 = load_dt(1);
+    float2 raw0 = load_dt(0), raw1 = load_dt(1);
     issue(0);
     issue(1);
     put_dt(0, raw0);
     put_dt(1, raw1);
-    float raw = load_dt(2);
+    float2 raw = load_dt(2);
     for (int gi = 0; gi < n_groups; ++gi) {
       asm volatile("cp.async.wait_group %0;" ::"n"(SS_STAGES - 2) : "memory");
       __syncthreads();                                   // stage gi has landed; stage gi - 1 is no longer read
@@ -152,31 +126,14 @@ ssd_scan_kernel(SsdArgs a) {
     return;
   }
   const int sub = lane & 15, lc = (warp * 2 + (lane >> 4)) * SS_CPL;       // the lane's rows; its first column in the block
-  const float skip = a.d_skip[h];
+  const float skip = a.d_skip != nullptr ? a.d_skip[h] : 0.f;
   // the state: rows 64 k + 4 sub + j of the lane's columns, in packed pairs
   f2 S[SS_CPL][2 * K4];
   float* st = a.state + ((size_t)slot * a.H + h) * P * N;
 #pragma unroll
   for (int c = 0; c < SS_CPL; ++c) {
     const int col = c0 + lc + c;
-    const float* sc = st + (size_t)col * N;
-#pragma unroll
-    for (int k = 0; k < K4; ++k) {
-      const int i = 64 * k + 4 * sub;
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (col < P) {
-        if constexpr (VEC) {
-          if (i < N) v = *reinterpret_cast<const float4*>(sc + i);
-        } else {
-          if (i < N) v.x = sc[i];
-          if (i + 1 < N) v.y = sc[i + 1];
-          if (i + 2 < N) v.z = sc[i + 2];
-          if (i + 3 < N) v.w = sc[i + 3];
-        }
-      }
-      S[c][2 * k] = pack_f2(v.x, v.y);
-      S[c][2 * k + 1] = pack_f2(v.z, v.w);
-    }
+    load_column<K4, VEC>(st + (size_t)col * N, N, sub, col < P, S[c]);
   }
   for (int gi = 0; gi < n_groups; ++gi) {
     __syncthreads();
@@ -259,20 +216,8 @@ ssd_scan_kernel(SsdArgs a) {
           }
         }
       }
-      // the run's 32 outputs of these four columns (number 4 tt + c), each the sum of 16 lanes' parts: in
-      // every round a lane hands half of its values over and adds the other half of its partner's, so that
-      // lane `sub` ends with the whole sums number 2 sub and 2 sub + 1
-      static_assert(SS_RUN * SS_CPL == 32, "two outputs per lane");
-#pragma unroll
-      for (int half = 16; half >= 2; half >>= 1) {
-        const bool upper = (lane & (half >> 1)) != 0;
-#pragma unroll
-        for (int i = 0; i < half; ++i) {
-          const float send = upper ? o[i] : o[i + half];
-          const float keep = upper ? o[i + half] : o[i];
-          o[i] = keep + __shfl_xor_sync(0xffffffffu, send, half >> 1);
-        }
-      }
+      // the run's 32 outputs of these four columns: lane `sub` gets those number 2 sub and 2 sub + 1
+      run_sums(o, lane);
       const int tt = first + (sub >> 1), lcc = lc + (sub & 1) * 2, col = c0 + lcc;
       if (tt < nt && col < P) {
         const float2 x = *reinterpret_cast<const float2*>(sg + tt * PER_TOK + 2 * NP + lcc);
@@ -290,23 +235,7 @@ ssd_scan_kernel(SsdArgs a) {
 #pragma unroll
   for (int c = 0; c < SS_CPL; ++c) {
     const int col = c0 + lc + c;
-    if (col >= P) continue;
-    float* sc = st + (size_t)col * N;
-#pragma unroll
-    for (int k = 0; k < K4; ++k) {
-      const int i = 64 * k + 4 * sub;
-      float4 v;
-      unpack_f2(S[c][2 * k], v.x, v.y);
-      unpack_f2(S[c][2 * k + 1], v.z, v.w);
-      if constexpr (VEC) {
-        if (i < N) *reinterpret_cast<float4*>(sc + i) = v;
-      } else {
-        if (i < N) sc[i] = v.x;
-        if (i + 1 < N) sc[i + 1] = v.y;
-        if (i + 2 < N) sc[i + 2] = v.z;
-        if (i + 3 < N) sc[i + 3] = v.w;
-      }
-    }
+    if (col < P) store_column<K4, VEC>(st + (size_t)col * N, N, sub, S[c]);
   }
 }
 
@@ -327,8 +256,10 @@ ssd_step_kernel(SsdArgs a) {
   float* st = a.state + ((size_t)slot * a.H + h) * P * N;
   const float* row = a.act + (size_t)t * (inner + 2 * a.G * N);
   pdl_wait();
-  const float dt = softplus(sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) + a.dt_bias[h]);
-  const float coef = decay_coef(-expf(a.a_log[h]) * dt), keep = decay_keep(coef);
+  const bool given = a.put != nullptr;
+  const float dt = given ? a.put[(size_t)t * a.H + h]
+                         : softplus(sum_slices(a.dt + (size_t)t * a.dt_row + h, a.dt_n, a.dt_stride) + a.dt_bias[h]);
+  const float coef = decay_coef(given ? a.log_decay[(size_t)t * a.H + h] : -expf(a.a_log[h]) * dt), keep = decay_keep(coef);
   float x[SD_COLS], y[SD_COLS];
 #pragma unroll
   for (int c = 0; c < SD_COLS; ++c) {
@@ -381,7 +312,7 @@ ssd_step_kernel(SsdArgs a) {
   y[0] += __shfl_xor_sync(0xffffffffu, y[0], 8);
   y[0] += __shfl_xor_sync(0xffffffffu, y[0], 16);
   if (lane < SD_COLS && c0 + lane < P)
-    a.out[(size_t)t * inner + h * P + c0 + lane] = fmaf(a.d_skip[h], row[h * P + c0 + lane], y[0]);
+    a.out[(size_t)t * inner + h * P + c0 + lane] = fmaf(a.d_skip != nullptr ? a.d_skip[h] : 0.f, row[h * P + c0 + lane], y[0]);
 }
 
 // grid (tokens, groups); y [tokens][inner]; z slices [z_n][tokens][z_row]; out [tokens][inner]
@@ -442,15 +373,18 @@ using namespace yalm;
 
 // act float32 [tokens][H P + 2 G N] = (x | B | C); dt: float32 slices whose column col0 + h is head h's raw
 // step; state float32 [slots][H][P][N], read at the step's start and written at its end; out float32
-// [tokens][H P].  N up to 256.
+// [tokens][H P].  N up to 256.  With put and log_decay float32 [tokens][H] those are dt_t and a_t themselves
+// (a_t <= 0), and dt, dt_bias, a_log are not read.  d_skip may be null.
 extern "C" int yalm_ssd_scan(const float* act, const float* dt, int dt_n, long long dt_stride, int dt_row, int col0,
-                             const float* dt_bias, const float* a_log, const float* d_skip, const int* q_start,
+                             const float* dt_bias, const float* a_log, const float* d_skip, const float* log_decay,
+                             const float* put, const int* q_start,
                              const int* seq_slot, float* state, float* out, int n_tokens, int n_seqs, int H, int G,
                              int P, int N, cudaStream_t stream) {
   if (n_seqs <= 0 || n_tokens <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || P <= 0 || N <= 0 || N > 256) return -2;
+  if ((put == nullptr) != (log_decay == nullptr) || (put == nullptr && (dt == nullptr || dt_bias == nullptr || a_log == nullptr))) return -3;
   if (n_seqs > 65535 || H > 65535) return -4;
-  const SsdArgs a = {act, dt + col0, dt_n, dt_row, dt_stride, dt_bias, a_log, d_skip, q_start, seq_slot, state, out, H, G, P, N};
+  const SsdArgs a = {act, dt + col0, dt_n, dt_row, dt_stride, dt_bias, a_log, d_skip, log_decay, put, q_start, seq_slot, state, out, H, G, P, N};
   const bool vec = N % 4 == 0 && P % 4 == 0 && ((((uintptr_t)act) | ((uintptr_t)state) | ((uintptr_t)out)) & 15) == 0;
   if (n_tokens == n_seqs) {                              // every sequence brings one token
     const dim3 sgrid((P + 8 * SD_COLS - 1) / (8 * SD_COLS), H, n_seqs), sblock(256);

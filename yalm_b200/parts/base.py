@@ -211,6 +211,7 @@ class ResidualStream:
         self.hold = False
         self.branches: list = []                       # (slices [S, N, D], S, norm weight | None, factor)
         self.branch_eps = 0.0
+        self.partials_name = "stream_partials"         # the buffer of a product's pending slices
         self.h: Optional[torch.Tensor] = None          # x in the compute type, while x is unchanged
         # A model that keeps several residual copies per token ("hyper-connections"): float32
         # [copies, N, D], made by ``spread``.  A sublayer's write into the copies is left here and
@@ -271,6 +272,10 @@ class ResidualStream:
         ``ops.norm_step`` takes it and y what the sublayer left on the held stream: the slices of its
         last product, or the scaled sum of a two-branch mixer's products.  Done by the next read."""
         self.settle()
+        self.due, self.h = (self.take_output(), form), None
+
+    def take_output(self) -> list:
+        """What the sublayer left on the held stream, as (slices, count, factor) sets whose sum is its output."""
         if self.branches:
             if any(w is not None for _, _, w, _ in self.branches):
                 raise RuntimeError("branches with norms of their own need a norm that sums them (sum_rmsnorm)")
@@ -281,7 +286,12 @@ class ResidualStream:
             self.pending, self.n_pending = None, 0
         else:
             raise RuntimeError("the sublayer left no output on the stream")
-        self.due, self.h = (sets, form), None
+        return sets
+
+    def leave_sum(self, sets) -> None:
+        """x <- x + the sum over ``sets`` (as ``ops.norm_step`` takes them), done by the next read."""
+        self.settle()
+        self.due, self.h = (list(sets), (ops.NORM_NONE, None, None, 0.0, 0.0)), None
 
     def settle(self) -> None:
         """Performs the write that ``post_norm`` left."""

@@ -196,3 +196,51 @@ class PrePostNormBlock:
         finally:
             stream.hold = False
         return later
+
+
+@register_block("parallel_prenorm")
+class ParallelPreNormBlock:
+    """Both sublayers read the same normed input, and one sum takes both outputs, each times a factor per
+    feature and a constant (``layer_scale`` parts): with h = norm(x),
+    x <- x + c_m w_m mixer(h) + c_f w_f ffn(h).  The parts are ``norm``, ``mixer``, ``mixer_scale``,
+    ``feed_forward``, ``feed_forward_scale`` (the last two may be absent).  The products stay apart from
+    x; the stream performs the whole sum together with the next norm's read, in one kernel."""
+
+    def __init__(self, layer_spec, rt):
+        self.spec = layer_spec
+        self.norm = make_part(NORMS, layer_spec.part("norm"), rt)
+        self.mixer = make_part(MIXERS, layer_spec.part("mixer"), rt)
+        self.mixer_scale = make_part(NORMS, layer_spec.part("mixer_scale"), rt)
+        self.ffn = self.ffn_scale = None
+        if "feed_forward" in layer_spec.parts:
+            self.ffn = make_part(FEED_FORWARDS, layer_spec.part("feed_forward"), rt)
+            self.ffn_scale = make_part(NORMS, layer_spec.part("feed_forward_scale"), rt)
+        for n in (self.mixer_scale, self.ffn_scale):
+            if n is not None and not hasattr(n, "scaled"):
+                raise TypeError("a parallel_prenorm block needs factors for its outputs (layer_scale)")
+
+    def parts(self):
+        s = self.spec
+        out = [(self.norm, s.part("norm")), (self.mixer, s.part("mixer")), (self.mixer_scale, s.part("mixer_scale"))]
+        if self.ffn is not None:
+            out += [(self.ffn, s.part("feed_forward")), (self.ffn_scale, s.part("feed_forward_scale"))]
+        return out
+
+    def mixers(self):
+        return {"mixer": self.mixer}
+
+    def forward(self, stream, batch, views, shared: bool = False):
+        stream.hold = True
+        try:
+            h = self.norm(stream)
+            later = self.mixer.forward(h, batch, stream, views["mixer"], shared=shared)
+            sets = self.mixer_scale.scaled(stream.take_output())
+            if self.ffn is not None:
+                stream.partials_name = "stream_partials_2"       # the mixer's slices are still to be read
+                self.ffn.forward(h, batch, stream)
+                sets += self.ffn_scale.scaled(stream.take_output())
+            stream.leave_sum(sets)
+        finally:
+            stream.hold = False
+            stream.partials_name = "stream_partials"
+        return later

@@ -126,6 +126,23 @@ def matmul_partials(rt, a: torch.Tensor, w: torch.Tensor, name: str) -> Tuple[to
     return buf, 1
 
 
+def stacked_rows(parts):
+    """(the matrices one below the other, the first row of each): projections of one input as one product.  All
+    are widened to 32 bits if one is stored so.  Parts start at multiples of four rows, and the whole has a
+    multiple of four (zero rows between and behind): the 16-byte loads of what reads the product's columns."""
+    if any(p.dtype == torch.float32 for p in parts):
+        parts = [p.to(torch.float32) for p in parts]
+    out, first, at = [], [], 0
+    for p in parts:
+        first.append(at)
+        out.append(p)
+        at += p.shape[0]
+        if at % 4:
+            out.append(torch.zeros((4 - at % 4, p.shape[1]), dtype=p.dtype, device=p.device))
+            at += 4 - at % 4
+    return torch.cat(out, 0), first
+
+
 def matmul_act(rt, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int, name: str) -> None:
     """out = act(a @ w.T), act one of ops.GELU_TANH / ops.TANH, applied to the 32-bit sums: many
     tokens in the two-SM product's epilogue (one launch, no 32-bit product in memory), few as
@@ -164,11 +181,11 @@ def matmul_into_stream(rt, a: torch.Tensor, w: torch.Tensor, stream) -> None:
             raise RuntimeError("the stream already holds a pending output")
         if _use_tc(rt, a, w) and M > MANY_TOKENS and plan_splits_many(M, N, K, rt.sm_count) > 1:
             S = plan_splits_many(M, N, K, rt.sm_count)       # few tiles: slices of K fill the idle pairs
-            buf = rt.buffer("stream_partials", (S, M, N), torch.float32)
+            buf = rt.buffer(stream.partials_name, (S, M, N), torch.float32)
             ops.gemm_2sm(a, w, buf, ops.GEMM_SPLIT, rt.status, splits=S)
             stream.pending, stream.n_pending = buf, S
         else:
-            stream.pending, stream.n_pending = matmul_partials(rt, a, w, "stream_partials")
+            stream.pending, stream.n_pending = matmul_partials(rt, a, w, stream.partials_name)
         return
     if stream.n_pending:
         stream.resolve()
@@ -176,13 +193,13 @@ def matmul_into_stream(rt, a: torch.Tensor, w: torch.Tensor, stream) -> None:
     if _use_tc(rt, a, w):
         if _small(rt, M, N):
             S = plan_splits(M, N, K, rt.sm_count)
-            buf = rt.buffer("stream_partials", (S, M, N), torch.float32)
+            buf = rt.buffer(stream.partials_name, (S, M, N), torch.float32)
             ops.gemm_tc(a, w, buf, ops.GEMM_SPLIT, rt.status, splits=S)
             stream.pending, stream.n_pending = buf, S
         elif M > MANY_TOKENS:
             S = plan_splits_many(M, N, K, rt.sm_count)
             if S > 1:
-                buf = rt.buffer("stream_partials", (S, M, N), torch.float32)
+                buf = rt.buffer(stream.partials_name, (S, M, N), torch.float32)
                 ops.gemm_2sm(a, w, buf, ops.GEMM_SPLIT, rt.status, splits=S)
                 stream.pending, stream.n_pending = buf, S
             else:

@@ -75,6 +75,28 @@ class LayerNorm:
         return stream.read_norm(self.form(), out, rows=rows, n_rows=n_rows)
 
 
+@register_norm("layer_scale")
+class LayerScale:
+    """Not a norm but what stands in its place behind a sublayer that is not normed: its output joins the
+    residual stream times a stored factor per feature and a constant, x <- x + factor * weight * y.  It
+    hands both to the block (``scaled``), which leaves the write to the stream's next read."""
+
+    def __init__(self, params: dict, rt):
+        self.rt = rt
+        self.size = int(params["size"])
+        self.factor = float(params.get("factor", 1.0))
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensor_needs(self):
+        return {"weight": TensorNeed((self.size,), init="ones")}
+
+    def bind(self, tensors) -> None:
+        self.weight = self.rt.vector(tensors["weight"])
+
+    def scaled(self, sets):
+        return [(buf, n, self.factor * f, self.weight) for buf, n, f in sets]
+
+
 @register_norm("dynamic_tanh")
 class DynamicTanh:
     """A norm that computes no mean and no variance: n(x) = tanh(alpha x) w + b, with a stored scalar
