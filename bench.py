@@ -520,7 +520,49 @@ SARALIX_SIZES = {
                       m_vdim=64, state=128, groups=8, norm_groups=8, ff=11008, experts=64, top=6, expert_ff=1792,
                       pattern="slm", vocab=32000),
 }
-DESIGNS = {"saralix": (SARALIX_SIZES, saralix_config, saralix_twin),
+def tetodra_config(width, heads, kv_heads, dim, vdim, b_heads, b_kv, b_dim, lin_heads, lin_dim, lin_vdim, mem_heads, mem_dim,
+                   mem_vdim, d_heads, d_kv, d_dim, d_vdim, ff, pattern, vocab):
+    """A Tetodra configuration with layers of the sizes a served model has (random weights): ``pattern`` is a
+    string of "2" (rotary attention beside gated linear attention), "p" (attention with a distance bias and
+    sinks beside the matrix memory) and "d" (the delta rule with one decay per head)."""
+    mlp = {"kind": "dense", "ff": ff}
+    layer = {"2": {"type": "parallel_2", "mlp": mlp,
+                   "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": float(dim) ** -0.5,
+                                      "rot": {"base": 5e5, "dims": dim}},
+                             "right": {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "tau": 16.0},
+                             "left_scale": 0.7, "right_scale": 0.7}},
+             "p": {"type": "parallel", "mlp": mlp,
+                   "mixer": {"left": {"heads": b_heads, "kv_heads": b_kv, "dim": b_dim, "vdim": b_dim, "scale": float(b_dim) ** -0.5,
+                                      "bias_max": 1024, "q_temp": {"coef": 0.1, "every": 8192}},
+                             "right": {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": 15.0},
+                             "left_scale": 0.7, "right_scale": 0.7}},
+             "d": {"type": "delta", "mlp": mlp,
+                   "mixer": {"heads": d_heads, "kv_heads": d_kv, "dim": d_dim, "vdim": d_vdim, "conv": 4}}}
+    return {"architecture": "Tetodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 1.0,
+            "embedding": {"scale": float(width) ** 0.5}, "layers": [layer[c] for c in pattern]}
+
+
+def tetodra_twin(width, heads, kv_heads, dim, vdim, b_heads, b_kv, b_dim, lin_heads, lin_dim, lin_vdim, mem_heads, mem_dim,
+                 mem_vdim, d_heads, d_kv, d_dim, d_vdim, ff, pattern, vocab):
+    """The closest model the library had before: the Llama / Mistral decoder with the same width, layers,
+    feed-forward and attention heads."""
+    return {"architectures": ["LlamaForCausalLM"], "hidden_size": width, "intermediate_size": ff,
+            "num_hidden_layers": len(pattern), "num_attention_heads": heads, "num_key_value_heads": kv_heads,
+            "head_dim": dim, "vocab_size": vocab, "max_position_embeddings": 32768, "rms_norm_eps": 1e-6,
+            "rope_theta": 500000.0, "tie_word_embeddings": True, "hidden_act": "silu", "bos_token_id": 1,
+            "eos_token_id": 2}
+
+
+TETODRA_SIZES = {
+    "w2048-2d2p": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=256, b_heads=16, b_kv=4, b_dim=128, lin_heads=8,
+                       lin_dim=128, lin_vdim=256, mem_heads=8, mem_dim=128, mem_vdim=256, d_heads=16, d_kv=8, d_dim=128,
+                       d_vdim=128, ff=5632, pattern="2d2p", vocab=32000),
+    "w4096-2dp": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, b_heads=32, b_kv=8, b_dim=128, lin_heads=16,
+                      lin_dim=128, lin_vdim=256, mem_heads=8, mem_dim=256, mem_vdim=512, d_heads=32, d_kv=16, d_dim=128,
+                      d_vdim=128, ff=11008, pattern="2dp", vocab=32000),
+}
+DESIGNS = {"tetodra": (TETODRA_SIZES, tetodra_config, tetodra_twin),
+           "saralix": (SARALIX_SIZES, saralix_config, saralix_twin),
            "samulorn": (SAMULORN_SIZES, samulorn_config, samulorn_twin),
            "golulix": (DESIGN_SIZES, golulix_config, dense_twin),
            "rudazen": (RUDAZEN_SIZES, rudazen_config, rudazen_twin),
@@ -671,7 +713,7 @@ def main():
                          "beside the dense decoder at equal sizes (random weights, a few layers)")
     ap.add_argument("--design", default="golulix", choices=sorted(DESIGNS),
                     help="with --compare-designs: which design runs beside the dense decoder")
-    ap.add_argument("--design-size", default=None, choices=sorted(set(DESIGN_SIZES) | set(RUDAZEN_SIZES) | set(NEKOTAR_SIZES) | set(SAMULORN_SIZES) | set(SARALIX_SIZES)),
+    ap.add_argument("--design-size", default=None, choices=sorted(name for sizes, _, _ in DESIGNS.values() for name in sizes),
                     help="with --compare-designs: one of the design's sizes instead of all")
     args = ap.parse_args()
 

@@ -91,9 +91,9 @@ def attend(q, k, v, past: int, scale: float, bias=None, sink=None):
     return torch.einsum("htk,khd->thd", e / den, v)
 
 
-def matrix_memory(q, k, v, i, f, S, n, m: float):
+def matrix_memory(q, k, v, i, f, S, n, m: float, pieces=None):
     """One head over T tokens: q, k [T, dk], v [T, dv], i, f [T] (logarithms); S [dk, dv], n [dk] changed in
-    place.  Returns (o [T, dv], the new m)."""
+    place.  Returns (o [T, dv], the new m); ``pieces``, a list, receives every token's S^T q, n.q and e^-m."""
     out = []
     for t in range(q.shape[0]):
         mt = max(float(f[t]) + m, float(i[t]))
@@ -101,6 +101,8 @@ def matrix_memory(q, k, v, i, f, S, n, m: float):
         S.mul_(keep).add_(put * torch.outer(k[t], v[t]))
         n.mul_(keep).add_(put * k[t])
         out.append(S.T @ q[t] / (max(abs(float(n @ q[t])), math.exp(-mt)) + 1e-6))
+        if pieces is not None:
+            pieces.append(torch.cat([S.T @ q[t], torch.stack([n @ q[t], q.new_tensor(math.exp(-mt))])]))
         m = mt
     return torch.stack(out), m
 
