@@ -14,7 +14,7 @@ import torch.nn.functional as F
 from plain_tetodra import (attend, delta_rule, distance_bucket, gated_linear, layer_norm, matrix_memory,
                            over_rms, query_temperature, rotate_halves, unit)
 from tetodra_helpers import (CONFIGS, NEEDLE, TOL, add_portions, needle_model, needle_tokens, plain_generate_greedy,
-                             plain_logits, random_tokens, weights_of)
+                             plain_logits, random_tokens, steady_tokens, weights_of)
 from trace_tools import (Trace, add_batches, add_tail, add_whole, compare, forced_decode, run_in_process,
                          run_trace_run)
 
@@ -452,7 +452,7 @@ def test_delta_rule_with_one_decay_per_head(ops, H, G, dk, dv):
         m = bt.n_tokens
         act = torch.full((m, ops.delta_head_row(H, G, dk, dv)), float("nan"), device=DEV)
         act[:, :C] = dev(act0[rows])
-        ops.delta_prep(act, dev(src[:, rows]), 2, col_b, 0, 0, None, H, G, dk, dv, head_decay=(col_a, dev(dt_bias), dev(a_log)))
+        ops.delta_head_prep(act, dev(src[:, rows]), 2, col_b, col_a, dev(dt_bias), dev(a_log), bt, H, G, dk, dv)
         out = torch.empty(m, H * dv, device=DEV)
         ops.delta_head_scan(act, bt, state, out, H, G, dk, dv)
         return out
@@ -491,7 +491,7 @@ def test_gated_heads(ops, heads, size):
 def test_residual_stream_layer_by_layer(name):
     cfg, seed = CONFIGS[name]
     w = weights_of(name)
-    toks = random_tokens(90, cfg["vocab"], seed + 5)
+    toks, _ = steady_tokens(name, 90, seed + 5)
     want = []
     ref = plain_logits(cfg, w, toks, taps=want)
     for dtype, tol in (("float32", 2e-5), ("bfloat16", 4e-2)):
@@ -514,8 +514,7 @@ def test_whole_tail_portions_batches(name, dtype):
     lengths = {"a": 150, "b": 1, "c": 66, "d": 23, "e": 129}           # across page borders (64, 128), one token
     reqs, refs = {}, {}
     for k, (rid, n) in enumerate(lengths.items()):
-        reqs[rid] = random_tokens(n, cfg["vocab"], seed * 10 + k)
-        refs[rid] = plain_logits(cfg, w, reqs[rid])
+        reqs[rid], refs[rid] = steady_tokens(name, n, seed * 10 + k)
     tr = Trace()
     add_whole(tr, reqs)
     add_tail(tr, {r: reqs[r] for r in ("a", "c", "d")}, tail=40)
@@ -572,8 +571,7 @@ def test_long_decoding_through_the_captured_step(name, dtype):
     w = weights_of(name)
     reqs, refs = {}, {}
     for k, (rid, n) in enumerate({"x": 240, "y": 90, "z": 141}.items()):
-        reqs[rid] = random_tokens(n, cfg["vocab"], seed * 7 + k)
-        refs[rid] = plain_logits(cfg, w, reqs[rid])
+        reqs[rid], refs[rid] = steady_tokens(name, n, seed * 7 + k)
     lm = _lm(cfg, w, dtype, max_context=256, max_batch=3)
     forced_decode(lm, reqs, {"x": 30, "y": 3, "z": 65}, refs, TOL[dtype])
     # the same slots again, other requests: nothing of the earlier states is left
@@ -623,8 +621,7 @@ def test_trace_replay_program(tmp_path):
     write_model(tmp_path / "model", cfg, w)
     reqs, refs = {}, {}
     for k, (rid, n) in enumerate({"a": 70, "b": 9}.items()):
-        reqs[rid] = random_tokens(n, cfg["vocab"], 50 + k)
-        refs[rid] = plain_logits(cfg, w, reqs[rid])
+        reqs[rid], refs[rid] = steady_tokens("tet_c", n, 50 + k)
     tr = Trace()
     add_whole(tr, reqs)
     add_tail(tr, reqs, tail=8)

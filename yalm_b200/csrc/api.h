@@ -419,10 +419,13 @@ int yalm_gated_rows(const float* z, int n_partials, long long partial_stride, co
 
 // ---- delta_rule.cu: the gated delta rule with a decay per key channel ------------------------------
 int yalm_delta_row(int H, int G, int dk, int dv);
-int yalm_delta_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row, int col_b,
-                    int col_low, int n_low, void* low, int low_dtype, int col_a, const float* dt_bias,
-                    const float* a_log, int n_tokens, int H, int G, int dk, int dv, cudaStream_t stream);
+int yalm_delta_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row,
+                    int col_b, int col_low, int n_low, void* low, int low_dtype, int n_tokens, int H, int G,
+                    int dk, int dv, cudaStream_t stream);
 int yalm_delta_head_row(int H, int G, int dk, int dv);
+int yalm_delta_head_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row, int col_b,
+                         int col_a, const float* dt_bias, const float* a_log, const int* q_start, int n_tokens, int n_seqs,
+                         int H, int G, int dk, int dv, cudaStream_t stream);
 int yalm_delta_head_scan(const float* act, const int* q_start, const int* seq_slot, float* state, float* out,
                          int n_tokens, int n_seqs, int H, int G, int dk, int dv, cudaStream_t stream);
 int yalm_delta_scan(float* act, const float* z, int n_partials, long long partial_stride,

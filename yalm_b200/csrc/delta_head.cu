@@ -1,26 +1,131 @@
 // The gated delta rule with ONE decay per head, per head with key size dk and value size dv:
 //   S <- e^(a_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t,   a_t <= 0
-// (delta_rule.cu has the form with a decay per key channel, and delta_prep, which makes the unit vectors, the
-// betas and the a_t).  32-bit throughout, the state carried from step to step as [slots][H][dv][dk]: a
-// column's rows are neighbours.
+// (delta_rule.cu has the form with a decay per key channel).  32-bit throughout, the state carried from step to
+// step as [slots][H][dv][dk]: a column's rows are neighbours.
 //
+// Tokens go in groups of 16.  With A_t = e^(a_first + .. + a_t) over a group and T = S / A the decay leaves the
+// elements, and the group's writes w_t (T <- T + k_t w_t^T) solve a triangular system whose matrix does not depend
+// on the state:
+//   w_t = beta_t (v_t / A_t - T_0^T k_t - sum_(s<t) (k_s.k_t) w_s),   o_t = A_t (T_0^T q_t + sum_(s<=t) (k_s.q_t) w_s)
+//   (I + L) w = beta r,  L_ts = beta_t (k_s.k_t) for s < t,  r_t = v_t / A_t - T_0^T k_t;   w = M r,  M = (I + L)^-1 beta
+// (the delta rule in this form: Yang et al., "Parallelizing Linear Transformers with the Delta Rule over Sequence
+// Length").  A group's reductions over the key channels are then made together, none waits for another's write.
+//
+//  * delta_head_prep: a block takes one group of one q/k head: q and k of every token become unit vectors
+//    (x / sqrt(sum x^2 + 1e-6)), q times 1/sqrt(dk); beta = sigmoid(.) and a = -exp(A_h) softplus(. + dt_h) for the
+//    heads that read it; and, for whole groups, the products k_s.q_t and every head's M.
 //  * delta_head_scan: a block owns 16 value columns of one (sequence, head), eight lanes own a column, a lane
-//    RPL of its rows in packed pairs; tokens come through a three-stage cp.async ring of 16.  With A_t =
-//    e^(a_first + .. + a_t) over a group of 16 tokens and T = S / A the decay leaves the elements:
-//        T <- T + k_t w^T,   w = beta_t (v_t / A_t - T^T k_t),   o_t = A_t T^T q_t,
-//    three multiply-adds per element and token, and S = A T at the group's end.  A group that forgets more
-//    than e^(-DH_SPAN) applies every token's own decay instead.  Every token needs one all-reduce over the
-//    eight lanes before its write; the outputs' sums are formed for 16 tokens at once.
+//    RPL of its rows in packed pairs; tokens come through a three-stage cp.async ring of 16.  Three multiply-adds
+//    per element and token.  A group that forgets more than e^(-DH_SPAN), and a sequence's last tokens, take the
+//    recurrence as it stands, one all-reduce over the eight lanes per token.
 //  * delta_head_step: one token per sequence, the state streamed once: a warp per DS_COLS columns.
 //
-// A token's row, float32: [q: G dk | k: G dk | v: H dv | beta: H padded to 4 | a: H padded to 4].
+// A token's row, float32: [q: G dk | k: G dk | v: H dv | beta: H padded to 4 | a: H padded to 4 | k_s.q_t: 16 G |
+// M's row: 16 H].
 #include "api.h"
 #include "scan.cuh"
 
 namespace yalm {
 
-constexpr int DH_TOK = 16, DH_STAGES = 3, DH_WARPS = 4, DH_COLS = 4 * DH_WARPS;
+constexpr int DH_TOK = SS_TOK, DH_STAGES = 3, DH_WARPS = 4, DH_COLS = 4 * DH_WARPS;
 constexpr float DH_SPAN = 30.f;
+
+struct DeltaHeadPrep {
+  float* act;
+  const float* proj;           // slices [n_partials][tokens][proj_row]: beta's logits at col_b, the decays' at col_a
+  int n_partials, proj_row, col_b, col_a;
+  long long partial_stride;
+  const float *dt_bias, *a_log;        // [H]
+  const int* q_start;
+  int n_seqs, row, H, G, dk, dv;
+};
+
+__device__ __forceinline__ int dh_tail(int H, int G, int dk, int dv) { return 2 * G * dk + H * dv + 2 * ((H + 3) & ~3); }
+
+constexpr int DP_THREADS = 128;
+
+// grid (groups of 16 tokens, q/k heads)
+__global__ void __launch_bounds__(DP_THREADS) delta_head_prep_kernel(DeltaHeadPrep a) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float dp_s[];         // q, k [16][pitch]; then betas [16][R], k.k [16][17]
+  int b, first;
+  if (!find_run<DH_TOK>(a.q_start, a.n_seqs, blockIdx.x, b, first)) return;
+  const int g = blockIdx.y, R = a.H / a.G, qs = a.q_start[b];
+  const int nt = min(DH_TOK, a.q_start[b + 1] - qs - first), t0 = qs + first;
+  const int pitch = ((a.dk + 3) & ~3) + 4, dkp = (a.dk + 3) & ~3;
+  float *q_s = dp_s, *k_s = q_s + DH_TOK * pitch, *beta_s = k_s + DH_TOK * pitch, *kk_s = beta_s + DH_TOK * R;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int beta0 = 2 * a.G * a.dk + a.H * a.dv, hp = (a.H + 3) & ~3, tail = dh_tail(a.H, a.G, a.dk, a.dv);
+  pdl_wait();
+  // 2 x 16 vectors over four warps: unit vectors, in memory and here
+  for (int i = warp; i < 2 * nt; i += DP_THREADS / 32) {
+    const int tt = i >> 1, is_k = i & 1;
+    float* v = a.act + (size_t)(t0 + tt) * a.row + (is_k * a.G + g) * a.dk;
+    float* d = (is_k ? k_s : q_s) + tt * pitch;
+    float x[8], ss = 0.f;                               // dk up to 256
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = lane + 32 * j;
+      x[j] = c < a.dk ? v[c] : 0.f;
+      ss += x[j] * x[j];
+    }
+    const float r = (1.0f / sqrtf(warp_sum(ss) + 1e-6f)) * (is_k ? 1.0f : 1.0f / sqrtf((float)a.dk));
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = lane + 32 * j;
+      if (c < a.dk) v[c] = x[j] * r;
+      if (c < dkp) d[c] = x[j] * r;                     // zero beyond dk
+    }
+  }
+  for (int i = threadIdx.x; i < nt * R; i += DP_THREADS) {
+    const int tt = i / R, r = i - tt * R, h = g * R + r;
+    const float* p = a.proj + (size_t)(t0 + tt) * a.proj_row + h;
+    float* o = a.act + (size_t)(t0 + tt) * a.row + beta0 + h;
+    const float beta = 1.0f / (1.0f + expf(-sum_slices(p + a.col_b, a.n_partials, a.partial_stride)));
+    const float z = sum_slices(p + a.col_a, a.n_partials, a.partial_stride) + a.dt_bias[h];
+    beta_s[tt * R + r] = beta;
+    o[0] = beta;
+    o[hp] = -expf(a.a_log[h]) * softplus(z);
+  }
+  if (nt < DH_TOK) return;                              // these tokens take the recurrence as it stands
+  __syncthreads();
+  {                                                     // token t = thread / 8 against s = 2 (thread % 8) and the next
+    const int t = threadIdx.x >> 3, s0 = (threadIdx.x & 7) * 2;
+    float kq[2] = {0.f, 0.f}, kk[2] = {0.f, 0.f};
+    for (int c = 0; c < dkp; c += 4) {
+      const float4 qt = *reinterpret_cast<const float4*>(q_s + t * pitch + c);
+      const float4 kt = *reinterpret_cast<const float4*>(k_s + t * pitch + c);
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const float4 ks = *reinterpret_cast<const float4*>(k_s + (s0 + j) * pitch + c);
+        kq[j] = fmaf(ks.x, qt.x, fmaf(ks.y, qt.y, fmaf(ks.z, qt.z, fmaf(ks.w, qt.w, kq[j]))));
+        kk[j] = fmaf(ks.x, kt.x, fmaf(ks.y, kt.y, fmaf(ks.z, kt.z, fmaf(ks.w, kt.w, kk[j]))));
+      }
+    }
+    float* o = a.act + (size_t)(t0 + t) * a.row + tail + g * DH_TOK + s0;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      o[j] = s0 + j <= t ? kq[j] : 0.f;
+      kk_s[t * 17 + s0 + j] = kk[j];
+    }
+  }
+  __syncthreads();
+  // a thread per (head, column s) of M
+  for (int i = threadIdx.x; i < R * DH_TOK; i += DP_THREADS) {
+    const int r = i / DH_TOK, s = i - r * DH_TOK;
+    float m[DH_TOK];
+    float* o = a.act + (size_t)t0 * a.row + tail + (a.G + g * R + r) * DH_TOK + s;
+    const float bs = beta_s[s * R + r];
+#pragma unroll
+    for (int t = 0; t < DH_TOK; ++t) {
+      float sum = 0.f;
+#pragma unroll
+      for (int u = 0; u < t; ++u) sum = fmaf(kk_s[t * 17 + u], m[u], sum);      // m[u] is 0 above the diagonal
+      m[t] = t < s ? 0.f : t == s ? 1.f : -beta_s[t * R + r] * sum;
+      o[(size_t)t * a.row] = m[t] * bs;
+    }
+  }
+}
 
 struct DeltaHead {
   const float* act;
@@ -30,11 +135,40 @@ struct DeltaHead {
   int row, H, G, dk, dv;
 };
 
+// The eight lanes' partial sums of a column's 16 values: in every round a lane hands half of its values to its
+// partner and adds the partner's other half to its own; lane `sub` is left with the whole sums number 2 sub and
+// 2 sub + 1 in v[0] and v[1]
+__device__ __forceinline__ void column_sums(float* v, int sub) {
+  static_assert(DH_TOK == 16, "two values per lane");
+#pragma unroll
+  for (int half = 4, n = 8; half >= 1; half >>= 1, n >>= 1) {
+    const bool upper = (sub & half) != 0;
+#pragma unroll
+    for (int i = 0; i < n; ++i) {
+      const float send = upper ? v[i] : v[i + n];
+      const float keep = upper ? v[i + n] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+    }
+  }
+}
+// a row of 16 numbers in shared memory times 16 in registers
+__device__ __forceinline__ float row_times(const float* row, const float* x) {
+  float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < DH_TOK; i += 4) {
+    const float4 m = *reinterpret_cast<const float4*>(row + i);
+    s[0] = fmaf(m.x, x[i], s[0]); s[1] = fmaf(m.y, x[i + 1], s[1]);
+    s[2] = fmaf(m.z, x[i + 2], s[2]); s[3] = fmaf(m.w, x[i + 3], s[3]);
+  }
+  return (s[0] + s[1]) + (s[2] + s[3]);
+}
+
 template <int RPL, int VEC>
-__global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHead a) {
+__global__ void __launch_bounds__(32 * DH_WARPS, 1) delta_head_scan_kernel(DeltaHead a) {
   pdl_launch_dependents();
   constexpr int DKP = 8 * RPL;                          // rows, padded
-  constexpr int PER_TOK = 2 * DKP + DH_COLS + 4;        // q, k, this block's v columns, beta, a (+ padding)
+  // q, k, this block's v columns, beta, a (+ padding), k_s.q_t, M's row
+  constexpr int OFF_S = 2 * DKP + DH_COLS, OFF_G = OFF_S + 4, PER_TOK = OFF_G + 2 * DH_TOK;
   constexpr int NT = 32 * DH_WARPS, NF = RPL / 2;
   extern __shared__ __align__(16) float dh_stage[];     // [DH_STAGES][DH_TOK][PER_TOK]
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * DH_COLS;
@@ -48,7 +182,8 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
     for (int i = threadIdx.x; i < DH_STAGES * DH_TOK * PER_TOK; i += NT) dh_stage[i] = 0.f;
     __syncthreads();
   }
-  const int per = (2 * dk + min(DH_COLS, dv - c0)) / VEC;
+  const int n_v = min(DH_COLS, dv - c0), per = (2 * dk + n_v + 2 * DH_TOK) / VEC;
+  const int tail = dh_tail(H, G, dk, dv);
   const int beta_off = 2 * G * dk + H * dv + h, hp = (H + 3) & ~3;
   pdl_wait();
   // register pair 2 j + e holds rows 4 (sub + 8 j) + 2 e and the next
@@ -83,12 +218,17 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
         int so, d;
         if (f < dk) { so = hq * dk + f; d = f; }
         else if (f < 2 * dk) { so = G * dk + hq * dk + (f - dk); d = DKP + (f - dk); }
-        else { so = 2 * G * dk + h * dv + c0 + (f - 2 * dk); d = 2 * DKP + (f - 2 * dk); }
-        for (int tt = 0; tt < nt; ++tt) ss_copy<4 * VEC>(dst + tt * PER_TOK + d, src + (size_t)tt * row + so);
+        else if (f < 2 * dk + n_v) { so = 2 * G * dk + h * dv + c0 + (f - 2 * dk); d = 2 * DKP + (f - 2 * dk); }
+        else {
+          const int e2 = f - 2 * dk - n_v;
+          so = tail + (e2 < DH_TOK ? hq * DH_TOK + e2 : (G + h) * DH_TOK + (e2 - DH_TOK));
+          d = OFF_G + e2;
+        }
+        ss_copy_tokens<4 * VEC>(dst + d, PER_TOK, src + so, row, nt);
       }
-      if (threadIdx.x < nt) ss_copy<4>(dst + threadIdx.x * PER_TOK + 2 * DKP + DH_COLS, src + (size_t)threadIdx.x * row + beta_off);
+      if (threadIdx.x < nt) ss_copy<4>(dst + threadIdx.x * PER_TOK + OFF_S, src + (size_t)threadIdx.x * row + beta_off);
       else if (threadIdx.x >= 32 && threadIdx.x < 32 + nt)
-        ss_copy<4>(dst + (threadIdx.x - 32) * PER_TOK + 2 * DKP + DH_COLS + 1, src + (size_t)(threadIdx.x - 32) * row + beta_off + hp);
+        ss_copy<4>(dst + (threadIdx.x - 32) * PER_TOK + OFF_S + 1, src + (size_t)(threadIdx.x - 32) * row + beta_off + hp);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -103,7 +243,7 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
     const float* sg = dh_stage + (size_t)(g % DH_STAGES) * DH_TOK * PER_TOK;
     // lane tt and lane 16 + tt of every warp: token tt's a and the sum up to it
     const int mine = lane & (DH_TOK - 1);
-    const float la = mine < nt ? sg[mine * PER_TOK + 2 * DKP + DH_COLS + 1] : -0.f;
+    const float la = mine < nt ? sg[mine * PER_TOK + OFF_S + 1] : -0.f;
     float cum = la;
 #pragma unroll
     for (int o = 1; o < DH_TOK; o <<= 1) {
@@ -125,7 +265,7 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
         qr[2 * j] = q2.x; qr[2 * j + 1] = q2.y;
         kr[2 * j] = k2.x; kr[2 * j + 1] = k2.y;
       }
-      const float beta = sg[tt * PER_TOK + 2 * DKP + DH_COLS];
+      const float beta = sg[tt * PER_TOK + OFF_S];
       float vj = sg[tt * PER_TOK + 2 * DKP + lc];
       const float fa = __shfl_sync(0xffffffffu, f_a, tt);
       if (scaled) {
@@ -164,9 +304,68 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
       o[tt] = (x0 + x1) + (x2 + x3);
       if (scaled) o[tt] *= fa;
     };
-    if (nt == DH_TOK && whole) {                        // the usual group: no test between the tokens
+    if (nt == DH_TOK && whole) {                        // the usual group
+      // T_0^T k_t and T_0^T q_t for all of its tokens, rows fetched one token ahead of their use
+      float kd[DH_TOK];
+      constexpr int NB = RPL <= 16 ? 2 : 1;
+      ulonglong2 qb[NB][RPL / 4], kb[NB][RPL / 4];
+      auto fetch = [&](int tt, bool q) {
+        const float* p = sg + tt * PER_TOK + 4 * sub;
 #pragma unroll
-      for (int tt = 0; tt < DH_TOK; ++tt) token(tt, true);
+        for (int j = 0; j < RPL / 4; ++j) {
+          kb[tt % NB][j] = *reinterpret_cast<const ulonglong2*>(p + DKP + 32 * j);
+          if (q) qb[tt % NB][j] = *reinterpret_cast<const ulonglong2*>(p + 32 * j);
+        }
+      };
+      if (NB == 2) fetch(0, true);
+#pragma unroll
+      for (int tt = 0; tt < DH_TOK; ++tt) {
+        if (NB == 1) fetch(tt, true);
+        else if (tt + 1 < DH_TOK) fetch(tt + 1, true);
+        const ulonglong2 *q2 = qb[tt % NB], *k2 = kb[tt % NB];
+        f2 k0 = mul_f2(k2[0].x, S[0]), k1 = mul_f2(k2[0].y, S[1]), q0 = mul_f2(q2[0].x, S[0]), q1 = mul_f2(q2[0].y, S[1]);
+#pragma unroll
+        for (int j = 1; j < RPL / 4; ++j) {
+          k0 = fma_f2(k2[j].x, S[2 * j], k0); k1 = fma_f2(k2[j].y, S[2 * j + 1], k1);
+          q0 = fma_f2(q2[j].x, S[2 * j], q0); q1 = fma_f2(q2[j].y, S[2 * j + 1], q1);
+        }
+        kd[tt] = sum_f2(k0, k1);
+        o[tt] = sum_f2(q0, q1);
+      }
+      // over the eight lanes; lane `sub` keeps those of tokens 2 sub and 2 sub + 1
+      column_sums(kd, sub);
+      column_sums(o, sub);
+      const float* mine_s = sg + (2 * sub) * PER_TOK;
+      float w[2], rr[DH_TOK];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        w[i] = fmaf(mine_s[i * PER_TOK + 2 * DKP + lc], __shfl_sync(0xffffffffu, f_inv, 2 * sub + i), -kd[i]);
+#pragma unroll
+      for (int tt = 0; tt < DH_TOK; ++tt) rr[tt] = __shfl_sync(0xffffffffu, w[tt & 1], (lane & 24) | (tt >> 1));
+#pragma unroll
+      for (int i = 0; i < 2; ++i) w[i] = row_times(mine_s + i * PER_TOK + OFF_G + DH_TOK, rr);
+#pragma unroll
+      for (int tt = 0; tt < DH_TOK; ++tt) rr[tt] = __shfl_sync(0xffffffffu, w[tt & 1], (lane & 24) | (tt >> 1));
+      // the outputs of this lane's two tokens, then the writes
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float A = __shfl_sync(0xffffffffu, f_a, 2 * sub + i);
+        const float y = A * (o[i] + row_times(mine_s + i * PER_TOK + OFF_G, rr));
+        if (col < dv) a.out[((size_t)(base + 2 * sub + i) * H + h) * dv + col] = y;
+      }
+      __syncwarp();                                     // the keys are loaded again, not kept in registers
+      if (NB == 2) fetch(0, false);
+#pragma unroll
+      for (int tt = 0; tt < DH_TOK; ++tt) {
+        if (NB == 1) fetch(tt, false);
+        else if (tt + 1 < DH_TOK) fetch(tt + 1, false);
+        const f2 ww = pack_f2(rr[tt], rr[tt]);
+#pragma unroll
+        for (int j = 0; j < RPL / 4; ++j) {
+          S[2 * j] = fma_f2(kb[tt % NB][j].x, ww, S[2 * j]);
+          S[2 * j + 1] = fma_f2(kb[tt % NB][j].y, ww, S[2 * j + 1]);
+        }
+      }
     } else if (whole) {
 #pragma unroll
       for (int tt = 0; tt < DH_TOK; ++tt) {
@@ -186,19 +385,8 @@ __global__ void __launch_bounds__(32 * DH_WARPS) delta_head_scan_kernel(DeltaHea
 #pragma unroll
       for (int r = 0; r < NF; ++r) S[r] = fma_f2(e, S[r], mul_f2(kp, S[r]));
     }
-    // the eight lanes' partial sums of the column's 16 outputs: in every round a lane hands half of its values to
-    // its partner and adds the partner's other half to its own; two whole sums are left per lane
-    static_assert(DH_TOK == 16, "two outputs per lane");
-#pragma unroll
-    for (int half = 4, n = 8; half >= 1; half >>= 1, n >>= 1) {
-      const bool upper = (sub & half) != 0;
-#pragma unroll
-      for (int i = 0; i < n; ++i) {
-        const float send = upper ? o[i] : o[i + n];
-        const float keep = upper ? o[i + n] : o[i];
-        o[i] = keep + __shfl_xor_sync(0xffffffffu, send, half);
-      }
-    }
+    if (nt == DH_TOK && whole) continue;
+    column_sums(o, sub);
     if (col < dv) {
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
@@ -321,9 +509,36 @@ __global__ void __launch_bounds__(256) delta_head_step_kernel(DeltaHead a) {
 using namespace yalm;
 
 // The length of a token's row (see the head of this file)
-extern "C" int yalm_delta_head_row(int H, int G, int dk, int dv) { return 2 * G * dk + H * dv + 2 * ((H + 3) & ~3); }
+extern "C" int yalm_delta_head_row(int H, int G, int dk, int dv) {
+  return 2 * G * dk + H * dv + 2 * ((H + 3) & ~3) + DH_TOK * (G + H);
+}
 
-// act float32 [tokens][yalm_delta_head_row]; state float32 [slots][H][dv][dk], read at the step's start and
+// act float32 [tokens][yalm_delta_head_row], whose first 2 G dk + H dv columns hold q | k | v after their convolution
+// and activation; proj: float32 slices [n_partials][tokens][proj_row] with the H beta logits at col_b and the H decay
+// logits at col_a; dt_bias, a_log [H].  dk up to 256.
+extern "C" int yalm_delta_head_prep(float* act, const float* proj, int n_partials, long long partial_stride, int proj_row,
+                                    int col_b, int col_a, const float* dt_bias, const float* a_log, const int* q_start,
+                                    int n_tokens, int n_seqs, int H, int G, int dk, int dv, cudaStream_t stream) {
+  if (n_tokens <= 0 || n_seqs <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || dk > 256) return -2;
+  if (G > 65535) return -4;
+  const DeltaHeadPrep a = {act, proj, n_partials, proj_row, col_b, col_a, partial_stride, dt_bias, a_log, q_start, n_seqs,
+                           yalm_delta_head_row(H, G, dk, dv), H, G, dk, dv};
+  const size_t smem = ((size_t)DH_TOK * 2 * (((dk + 3) & ~3) + 4) + (size_t)DH_TOK * (H / G) + DH_TOK * 17) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  static size_t attr = 48 * 1024;
+  if (smem > attr) {
+    cudaError_t e = cudaFuncSetAttribute(delta_head_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    attr = smem;
+  }
+  const int runs = n_tokens == n_seqs ? n_tokens : n_tokens / DH_TOK + n_seqs;
+  launch_pdl(delta_head_prep_kernel, dim3(runs, G), dim3(DP_THREADS), smem, stream, a);
+  YALM_LAUNCH_CHECK();
+  return 0;
+}
+
+// act as delta_head_prep leaves it; state float32 [slots][H][dv][dk], read at the step's start and
 // written at its end; out float32 [tokens][H dv].  dk up to 256.
 extern "C" int yalm_delta_head_scan(const float* act, const int* q_start, const int* seq_slot, float* state, float* out,
                                     int n_tokens, int n_seqs, int H, int G, int dk, int dv, cudaStream_t stream) {
@@ -344,7 +559,7 @@ extern "C" int yalm_delta_head_scan(const float* act, const int* q_start, const 
   const dim3 grid((dv + DH_COLS - 1) / DH_COLS, H, n_seqs), block(32 * DH_WARPS);
 #define YALM_DH1(R, V)                                                                                             \
   do {                                                                                                             \
-    const size_t smem = (size_t)DH_STAGES * DH_TOK * (2 * 8 * R + DH_COLS + 4) * sizeof(float);                    \
+    const size_t smem = (size_t)DH_STAGES * DH_TOK * (2 * 8 * R + DH_COLS + 4 + 2 * DH_TOK) * sizeof(float);                    \
     static bool set = false;                                                                                       \
     if (!set && smem > 48 * 1024) {                                                                                \
       cudaError_t e = cudaFuncSetAttribute(delta_head_scan_kernel<R, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \

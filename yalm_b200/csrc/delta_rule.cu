@@ -5,8 +5,7 @@
 //
 //  * delta_prep: q and k of every token and q/k head become unit vectors (x / sqrt(sum x^2 + 1e-6)),
 //    q times 1/sqrt(dk); beta = sigmoid(.); and the two low-rank projections' first halves go out in
-//    the storage type as the input of their second halves (or, for the form with one decay per head of
-//    delta_head.cu, the decays' logarithms -exp(A_h) softplus(. + dt_h));
+//    the storage type as the input of their second halves;
 //  * delta_decay: the decay per head and key channel, kept as g - 1 = expm1(-exp(A_h) softplus(z + dt))
 //    (a decay close to 1 has few bits of its own left in g; S + (g - 1) S keeps them), and the output
 //    gate sigmoid(.) per head and value channel;
@@ -35,9 +34,7 @@ __device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log
 template <typename T>
 __global__ void delta_prep_kernel(float* __restrict__ act, int row, const float* __restrict__ proj,
                                   int n_partials, long long partial_stride, int proj_row, int col_b,
-                                  int col_low, int n_low, T* __restrict__ low, int col_a,
-                                  const float* __restrict__ dt_bias, const float* __restrict__ a_log, int H, int G,
-                                  int dk, int dv) {
+                                  int col_low, int n_low, T* __restrict__ low, int H, int G, int dk, int dv) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -57,10 +54,6 @@ __global__ void delta_prep_kernel(float* __restrict__ act, int row, const float*
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     const float z = sum_slices(p + col_b + i, n_partials, partial_stride);
     a[beta0 + i] = 1.0f / (1.0f + expf(-z));
-    if (a_log != nullptr) {                                 // one decay per head: its logarithm, after the betas
-      const float d = sum_slices(p + col_a + i, n_partials, partial_stride);
-      a[beta0 + ((H + 3) & ~3) + i] = -expf(a_log[i]) * softplus_f(d + dt_bias[i]);
-    }
   }
   for (int i = threadIdx.x; i < n_low; i += blockDim.x)
     low[(size_t)t * n_low + i] = from_float<T>(sum_slices(p + col_low + i, n_partials, partial_stride));
@@ -423,22 +416,20 @@ extern "C" int yalm_delta_row(int H, int G, int dk, int dv) {
   return 2 * G * dk + H * dv + ((H + 3) & ~3) + H * dk;
 }
 
-// act: float32 [tokens][row], whose first 2 G dk + H dv columns hold q | k | v after their
+// act: float32 [tokens][yalm_delta_row], whose first 2 G dk + H dv columns hold q | k | v after their
 // convolution and activation.  proj: slices [.][tokens][proj_row] of the mixer's first product, with
 // the beta logits at column col_b and the n_low low-rank values at col_low; low [tokens][n_low] in
-// low_dtype receives those.  With a_log and dt_bias [H] the decay logits, one per head, are at column col_a
-// and row is yalm_delta_head_row; else row is yalm_delta_row.
+// low_dtype receives those.
 extern "C" int yalm_delta_prep(float* act, const float* proj, int n_partials, long long partial_stride,
                                int proj_row, int col_b, int col_low, int n_low, void* low, int low_dtype,
-                               int col_a, const float* dt_bias, const float* a_log,
                                int n_tokens, int H, int G, int dk, int dv, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || n_low < 0 || (a_log != nullptr && dt_bias == nullptr)) return -2;
-  const int row = a_log != nullptr ? yalm_delta_head_row(H, G, dk, dv) : yalm_delta_row(H, G, dk, dv);
+  if (H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || n_low < 0) return -2;
+  const int row = yalm_delta_row(H, G, dk, dv);
   const dim3 grid(n_tokens), block(256);
 #define YALM_DP(T)                                                                                     \
   launch_pdl(delta_prep_kernel<T>, grid, block, 0, stream, act, row, proj, n_partials, partial_stride, \
-             proj_row, col_b, col_low, n_low, (T*)low, col_a, dt_bias, a_log, H, G, dk, dv)
+             proj_row, col_b, col_low, n_low, (T*)low, H, G, dk, dv)
   if (low_dtype == DT_F32) YALM_DP(float);
   else if (low_dtype == DT_BF16) YALM_DP(__nv_bfloat16);
   else if (low_dtype == DT_F16) YALM_DP(__half);

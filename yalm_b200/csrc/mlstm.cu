@@ -34,7 +34,19 @@ struct MlstmPrep {
 
 constexpr int ML_THREADS = 256;
 
-// blocks 0 .. n_seqs H - 1: a (sequence, head)'s gates; the others: 1,024 elements of one token's row
+__device__ __forceinline__ float4 four_of(const float* p, int n, long long stride) {
+  float4 v = *reinterpret_cast<const float4*>(p);
+  for (int k = 1; k < n; ++k) {
+    const float4 u = *reinterpret_cast<const float4*>(p + (size_t)k * stride);
+    v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+  }
+  return v;
+}
+
+// blocks 0 .. n_seqs H - 1: a (sequence, head)'s gates; the others: ML_PART elements of one token's row.  VEC: sizes,
+// columns and pointers allow 16-byte accesses
+constexpr int ML_PART = 2048;
+template <bool VEC>
 __global__ void __launch_bounds__(ML_THREADS) mlstm_prep_kernel(MlstmPrep a, int parts) {
   pdl_launch_dependents();
   const int n_gate = a.n_seqs * a.H;
@@ -44,18 +56,38 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_prep_kernel(MlstmPrep a, int
     pdl_wait();
     const float* p = a.proj + (size_t)t * a.proj_row;
     float* o = a.act + (size_t)t * row;
-    const int end = min(row, (part + 1) * 1024);
-    for (int e = part * 1024 + threadIdx.x; e < end; e += ML_THREADS) {
-      float v;
-      if (e < n_x) {
-        const int h = e / a.P, c = e - h * a.P;
-        v = c < a.dv ? sum_slices(p + a.col_v + h * a.dv + c, a.n_partials, a.partial_stride) : (c == a.dv ? 1.f : 0.f);
-      } else if (e < n_x + n_k) {
-        v = sum_slices(p + a.col_k + (e - n_x), a.n_partials, a.partial_stride);
-      } else {
-        v = sum_slices(p + a.col_q + (e - n_x - n_k), a.n_partials, a.partial_stride) * a.q_scale;
+    const int end = min(row, (part + 1) * ML_PART);
+    if constexpr (VEC) {
+#pragma unroll
+      for (int u = 0; u < ML_PART / (4 * ML_THREADS); ++u) {
+        const int e = part * ML_PART + (u * ML_THREADS + threadIdx.x) * 4;
+        if (e >= end) continue;
+        float4 v;
+        if (e < n_x) {
+          const int h = e / a.P, c = e - h * a.P;
+          v = c < a.dv ? four_of(p + a.col_v + h * a.dv + c, a.n_partials, a.partial_stride)
+                       : make_float4(c == a.dv ? 1.f : 0.f, 0.f, 0.f, 0.f);
+        } else if (e < n_x + n_k) {
+          v = four_of(p + a.col_k + (e - n_x), a.n_partials, a.partial_stride);
+        } else {
+          v = four_of(p + a.col_q + (e - n_x - n_k), a.n_partials, a.partial_stride);
+          v.x *= a.q_scale; v.y *= a.q_scale; v.z *= a.q_scale; v.w *= a.q_scale;
+        }
+        *reinterpret_cast<float4*>(o + e) = v;
       }
-      o[e] = v;
+    } else {
+      for (int e = part * ML_PART + threadIdx.x; e < end; e += ML_THREADS) {
+        float v;
+        if (e < n_x) {
+          const int h = e / a.P, c = e - h * a.P;
+          v = c < a.dv ? sum_slices(p + a.col_v + h * a.dv + c, a.n_partials, a.partial_stride) : (c == a.dv ? 1.f : 0.f);
+        } else if (e < n_x + n_k) {
+          v = sum_slices(p + a.col_k + (e - n_x), a.n_partials, a.partial_stride);
+        } else {
+          v = sum_slices(p + a.col_q + (e - n_x - n_k), a.n_partials, a.partial_stride) * a.q_scale;
+        }
+        o[e] = v;
+      }
     }
     return;
   }
@@ -204,12 +236,15 @@ extern "C" int yalm_mlstm_prep(const float* proj, int n_partials, long long part
                                int dk, int dv, int P, cudaStream_t stream) {
   if (n_tokens <= 0 || n_seqs <= 0) return 0;
   if (H <= 0 || dk <= 0 || dv <= 0 || P <= dv || !(cap > 0.f)) return -2;
-  const int parts = (H * P + 2 * H * dk + 1023) / 1024;
+  const int parts = (H * P + 2 * H * dk + ML_PART - 1) / ML_PART;
   const long long blocks = (long long)n_seqs * H + (long long)n_tokens * parts;
   if (blocks > 0x7fffffffLL) return -4;
   const MlstmPrep a = {proj, n_partials, proj_row, col_q, col_k, col_v, col_i, col_f, partial_stride, i_bias, f_bias,
                        act, log_decay, put, floor, maxima, q_start, seq_slot, n_tokens, n_seqs, H, dk, dv, P, cap, q_scale};
-  launch_pdl(mlstm_prep_kernel, dim3((unsigned)blocks), dim3(ML_THREADS), 0, stream, a, parts);
+  const bool vec = dk % 4 == 0 && dv % 4 == 0 && P % 4 == 0 && proj_row % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 &&
+                   col_v % 4 == 0 && (partial_stride & 3) == 0 && ((((uintptr_t)proj) | ((uintptr_t)act)) & 15) == 0;
+  if (vec) launch_pdl(mlstm_prep_kernel<true>, dim3((unsigned)blocks), dim3(ML_THREADS), 0, stream, a, parts);
+  else launch_pdl(mlstm_prep_kernel<false>, dim3((unsigned)blocks), dim3(ML_THREADS), 0, stream, a, parts);
   YALM_LAUNCH_CHECK();
   return 0;
 }

@@ -134,6 +134,7 @@ _SIGNATURES = {
     "yalm_head_store": [_vp, _i, _ll, _vp, _vp, _f, _i, _vp, _i, _f, _f] + [_vp] * 8 + [_i] * 9 + [_vp, _i, _i, _vp],
     "yalm_attention_kv": [_vp] * 9 + [_i] * 9 + [_f, _vp, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _vp],
     "yalm_delta_head_row": [_i, _i, _i, _i],
+    "yalm_delta_head_prep": [_vp, _vp, _i, _ll, _i, _i, _i, _vp, _vp, _vp] + [_i] * 6 + [_vp],
     "yalm_delta_head_scan": [_vp] * 5 + [_i] * 6 + [_vp],
     "yalm_gated_group_norm": [_vp, _vp, _i, _ll, _i, _i, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "yalm_activation_rows": [_vp, _i, _ll, _vp, _i, _ll, _i, _vp],
@@ -143,7 +144,7 @@ _SIGNATURES = {
                         _i, _i, _i, _i, _i, _vp],
     "yalm_gated_rows": [_vp, _i, _ll, _vp, _vp, _i, _i, _i, _vp, _i, _i, _i, _vp],
     "yalm_delta_row": [_i, _i, _i, _i],
-    "yalm_delta_prep": [_vp, _vp, _i, _ll, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "yalm_delta_prep": [_vp, _vp, _i, _ll, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "yalm_delta_scan": [_vp, _vp, _i, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "yalm_rglru": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _ll, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
                    _f, _vp],
@@ -1293,10 +1294,27 @@ def delta_head_row(H: int, G: int, dk: int, dv: int) -> int:
     return int(lib().yalm_delta_head_row(H, G, dk, dv))
 
 
+def delta_head_prep(act: torch.Tensor, proj: torch.Tensor, n_partials: int, col_b: int, col_a: int,
+                    dt_bias: torch.Tensor, a_log: torch.Tensor, batch, H: int, G: int, dk: int, dv: int) -> None:
+    """act float32 [N, delta_head_row] holds q | k | v (after convolution and SiLU) in its first columns: q and k
+    become unit vectors per head (q also times dk^-1/2); beta = sigmoid of the H columns of ``proj`` (float32
+    slices [(s,) N, row]) from col_b, the decays' logarithms -exp(a_log) softplus(the H columns from col_a +
+    dt_bias), and what ``delta_head_scan`` reads of every whole group of 16 tokens."""
+    n, row = batch.n_tokens, proj.shape[-1]
+    _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, delta_head_row(H, G, dk, dv))
+          and proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[-2] == n
+          and max(col_b, col_a) + H <= row, "delta_head_prep: shapes")
+    for v in (dt_bias, a_log):
+        _need(v.dtype == torch.float32 and v.numel() == H, "delta_head_prep: dt_bias, a_log float32 [H]")
+    _check(lib().yalm_delta_head_prep(_p(act), _p(proj), int(n_partials), n * row, row, int(col_b), int(col_a), _p(dt_bias),
+                                      _p(a_log), _p(batch.q_start), n, batch.n_seqs, H, G, dk, dv, _stream()),
+           "delta_head_prep")
+
+
 def delta_head_scan(act: torch.Tensor, batch, state: torch.Tensor, out: torch.Tensor, H: int, G: int, dk: int,
                     dv: int) -> None:
-    """The gated delta rule with one decay per head over the step's tokens: act float32 [N, delta_head_row] = (q |
-    k | v | beta | log decay), state float32 [slots, H, dv, dk], out float32 [N, H dv]."""
+    """The gated delta rule with one decay per head over the step's tokens: act float32 [N, delta_head_row] as
+    ``delta_head_prep`` leaves it, state float32 [slots, H, dv, dk], out float32 [N, H dv]."""
     n = batch.n_tokens
     _need(act.dtype == torch.float32 and act.is_contiguous() and tuple(act.shape) == (n, delta_head_row(H, G, dk, dv))
           and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dv, dk)
@@ -1430,24 +1448,19 @@ def delta_row(H: int, G: int, dk: int, dv: int) -> int:
 
 
 def delta_prep(act: torch.Tensor, proj: torch.Tensor, n_partials: int, col_b: int, col_low: int, n_low: int,
-               low: Optional[torch.Tensor], H: int, G: int, dk: int, dv: int, head_decay=None) -> None:
+               low: torch.Tensor, H: int, G: int, dk: int, dv: int) -> None:
     """act float32 [N, delta_row] holds q | k | v (after convolution and SiLU) in its first columns: q and
     k become unit vectors per head (q also times dk^-1/2), beta = sigmoid of the H columns of ``proj``
     (float32 slices [(s,) N, row]) from col_b, and the n_low columns from col_low go to ``low`` [N, n_low]
-    in low's type.  ``head_decay`` = (column of the H decay logits, dt_bias [H], a_log [H]): the rows are
-    those of ``delta_head_scan`` and receive the logarithms of the decays."""
+    in low's type."""
     n = act.shape[0]
-    want = delta_row(H, G, dk, dv) if head_decay is None else delta_head_row(H, G, dk, dv)
-    _need(act.dtype == torch.float32 and act.is_contiguous() and act.shape[1] == want
+    _need(act.dtype == torch.float32 and act.is_contiguous() and act.shape[1] == delta_row(H, G, dk, dv)
           and proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[-2] == n
-          and (n_low == 0 or (low.is_contiguous() and tuple(low.shape) == (n, n_low))), "delta_prep: shapes")
-    col_a, dt_bias, a_log = head_decay if head_decay is not None else (0, None, None)
-    for v in (dt_bias, a_log):
-        _need(v is None or (v.dtype == torch.float32 and v.numel() == H), "delta_prep: dt_bias, a_log float32 [H]")
+          and low.is_contiguous() and tuple(low.shape) == (n, n_low), "delta_prep: shapes")
     row = proj.shape[-1]
     _check(lib().yalm_delta_prep(_p(act), _p(proj), int(n_partials), n * row, row, int(col_b), int(col_low),
-                                 int(n_low), _p(low), dtype_code(low.dtype) if low is not None else F32, int(col_a),
-                                 _p(dt_bias), _p(a_log), n, H, G, dk, dv, _stream()), "delta_prep")
+                                 int(n_low), _p(low), dtype_code(low.dtype), n, H, G, dk, dv, _stream()),
+           "delta_prep")
 
 
 def delta_scan(act: torch.Tensor, z: torch.Tensor, n_partials: int, dt_bias: torch.Tensor, a_log: torch.Tensor,

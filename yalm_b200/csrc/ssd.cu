@@ -4,8 +4,8 @@
 //   dt_t = softplus(raw_t + bias),   a_t = -exp(A_log) dt_t,
 // B and C shared by the heads of a group.  Everything here is 32-bit.  Three kernels:
 //
-//  * ssd_scan: a block owns SS_COLS = 32 value columns of one (sequence, head).  The columns of S are
-//    independent; 16 lanes own SS_CPL = 4 of them, a lane 4 K4 rows of those, in packed pairs (two FP32
+//  * ssd_scan: a block owns 32 (or 16) value columns of one (sequence, head).  The columns of S are
+//    independent; 16 lanes own CPL = 4 (or 2) of them, a lane 4 K4 rows of those, in packed pairs (two FP32
 //    operations per instruction).  Four warps compute; a fifth feeds them: it brings the tokens (B | C |
 //    the block's x) through a three-stage cp.async ring of SS_TOK and turns their raw steps into dt and
 //    decays.  The sums over the 16 lanes are formed for SS_RUN tokens at once.  Runs of SS_RUN whole
@@ -43,23 +43,24 @@ struct SsdArgs {
 };
 
 // K4: groups of four rows per lane (64 K4 >= N); VEC: N, P and the pointers allow 16-byte accesses
-template <int K4, bool VEC>
-__global__ void __launch_bounds__(160)
+template <int K4, bool VEC, int CPL>
+__global__ void __launch_bounds__(160, 1)
 ssd_scan_kernel(SsdArgs a) {
   pdl_launch_dependents();
+  constexpr int COLS = 8 * CPL;
   constexpr int NP = 64 * K4;                            // rows, padded
-  constexpr int PER_TOK = 2 * NP + SS_COLS;              // B, C, then this block's x columns
+  constexpr int PER_TOK = 2 * NP + COLS;              // B, C, then this block's x columns
   extern __shared__ __align__(16) float ss_stage[];      // [SS_STAGES][SS_TOK][PER_TOK]
   // per token: the decay's coefficient, dt, and for whole runs A_t and dt / A_t
   __shared__ __align__(16) float4 step_s[SS_STAGES][SS_TOK];
   __shared__ float2 run_s[SS_STAGES][SS_TOK / SS_RUN];   // a run's sum of a, its decay's coefficient
-  const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * SS_COLS;
+  const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int slot = a.seq_slot[b];
   const int t0 = a.q_start[b], t1 = a.q_start[b + 1];
   const int N = a.N, P = a.P, inner = a.H * P;
   // rows beyond N and columns beyond P: never copied over, zero for ever
-  if (N < NP || c0 + SS_COLS > P) {
+  if (N < NP || c0 + COLS > P) {
     for (int i = threadIdx.x; i < SS_STAGES * SS_TOK * PER_TOK; i += blockDim.x) ss_stage[i] = 0.f;
     __syncthreads();
   }
@@ -70,7 +71,7 @@ ssd_scan_kernel(SsdArgs a) {
     const bool given = a.put != nullptr;
     const float neg_a = given ? 0.f : -expf(a.a_log[h]), bias = given ? 0.f : a.dt_bias[h];
     constexpr int W = VEC ? 4 : 1;
-    const int per = (2 * N + min(SS_COLS, P - c0)) / W;  // copies per token
+    const int per = (2 * N + min(COLS, P - c0)) / W;  // copies per token
     auto issue = [&](int gi) {
       if (gi < n_groups) {
         const int base = t0 + gi * SS_TOK;
@@ -83,7 +84,7 @@ ssd_scan_kernel(SsdArgs a) {
           else if (f < 2 * N) { so = inner + (a.G + g) * N + (f - N); d = NP + (f - N); }
           else { so = h * P + c0 + (f - 2 * N); d = 2 * NP + (f - 2 * N); }
           const float* src = a.act + (size_t)base * row + so;
-          for (int tt = 0; tt < nt; ++tt) ss_copy<4 * W>(dst + tt * PER_TOK + d, src + (size_t)tt * row);
+          ss_copy_tokens<4 * W>(dst + d, PER_TOK, src, row, nt);
         }
       }
       asm volatile("cp.async.commit_group;" ::: "memory");
@@ -125,13 +126,13 @@ ssd_scan_kernel(SsdArgs a) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     return;
   }
-  const int sub = lane & 15, lc = (warp * 2 + (lane >> 4)) * SS_CPL;       // the lane's rows; its first column in the block
+  const int sub = lane & 15, lc = (warp * 2 + (lane >> 4)) * CPL;       // the lane's rows; its first column in the block
   const float skip = a.d_skip != nullptr ? a.d_skip[h] : 0.f;
   // the state: rows 64 k + 4 sub + j of the lane's columns, in packed pairs
-  f2 S[SS_CPL][2 * K4];
+  f2 S[CPL][2 * K4];
   float* st = a.state + ((size_t)slot * a.H + h) * P * N;
 #pragma unroll
-  for (int c = 0; c < SS_CPL; ++c) {
+  for (int c = 0; c < CPL; ++c) {
     const int col = c0 + lc + c;
     load_column<K4, VEC>(st + (size_t)col * N, N, sub, col < P, S[c]);
   }
@@ -146,60 +147,51 @@ ssd_scan_kernel(SsdArgs a) {
       const int first = r * SS_RUN;
       if (first >= nt) break;
       const float2 run = run_s[gi % SS_STAGES][r];
-      float o[SS_RUN * SS_CPL];
+      float o[SS_RUN * CPL];
       if (nt >= first + SS_RUN && run.x >= -SS_SPAN) {
+        RunToken<K4, CPL> buf[2];
+        auto fetch = [&](int tt) {
+          const float* p = sg + (first + tt) * PER_TOK;
+          buf[tt & 1].fetch(p + NP + 4 * sub, p + 4 * sub, p + 2 * NP + lc);
+        };
+        fetch(0);
 #pragma unroll
         for (int tt = 0; tt < SS_RUN; ++tt) {
-          const float* p = sg + (first + tt) * PER_TOK;
           const float4 sv = steps[first + tt];
-          const float4 xv = *reinterpret_cast<const float4*>(p + 2 * NP + lc);
-          const float x[SS_CPL] = {sv.w * xv.x, sv.w * xv.y, sv.w * xv.z, sv.w * xv.w};
-          f2 oc[SS_CPL];
+          if (tt + 1 < SS_RUN) fetch(tt + 1);
 #pragma unroll
-          for (int k = 0; k < K4; ++k) {
-            const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(p + 64 * k + 4 * sub);
-            const ulonglong2 C = *reinterpret_cast<const ulonglong2*>(p + NP + 64 * k + 4 * sub);
+          for (int c = 0; c < CPL; ++c) buf[tt & 1].x[c] *= sv.w;
+          buf[tt & 1].apply(S, o + CPL * tt);
 #pragma unroll
-            for (int c = 0; c < SS_CPL; ++c) {
-              const f2 xd = pack_f2(x[c], x[c]);
-              S[c][2 * k] = fma_f2(B.x, xd, S[c][2 * k]);
-              S[c][2 * k + 1] = fma_f2(B.y, xd, S[c][2 * k + 1]);
-              oc[c] = k == 0 ? mul_f2(S[c][0], C.x) : fma_f2(S[c][2 * k], C.x, oc[c]);
-              oc[c] = fma_f2(S[c][2 * k + 1], C.y, oc[c]);
-            }
-          }
-#pragma unroll
-          for (int c = 0; c < SS_CPL; ++c) {
-            float lo, hi;
-            unpack_f2(oc[c], lo, hi);
-            o[SS_CPL * tt + c] = sv.z * (lo + hi);
-          }
+          for (int c = 0; c < CPL; ++c) o[CPL * tt + c] *= sv.z;
         }
         const float keep = decay_keep(run.y);
         const f2 e = pack_f2(run.y, run.y), kp = pack_f2(keep, keep);
 #pragma unroll
-        for (int c = 0; c < SS_CPL; ++c)
+        for (int c = 0; c < CPL; ++c)
 #pragma unroll
           for (int k = 0; k < 2 * K4; ++k) S[c][k] = fma_f2(e, S[c][k], mul_f2(kp, S[c][k]));
       } else {
 #pragma unroll
         for (int tt = 0; tt < SS_RUN; ++tt) {
 #pragma unroll
-          for (int c = 0; c < SS_CPL; ++c) o[SS_CPL * tt + c] = 0.f;
+          for (int c = 0; c < CPL; ++c) o[CPL * tt + c] = 0.f;
           if (first + tt < nt) {
             const float* p = sg + (first + tt) * PER_TOK;
             const float4 sv = steps[first + tt];
             const float keep = decay_keep(sv.x);
             const f2 am = pack_f2(sv.x, sv.x), kp = pack_f2(keep, keep);
-            const float4 xv = *reinterpret_cast<const float4*>(p + 2 * NP + lc);
-            const float x[SS_CPL] = {sv.y * xv.x, sv.y * xv.y, sv.y * xv.z, sv.y * xv.w};
-            f2 oc[SS_CPL];
+            float x[CPL];
+            load_columns<CPL>(p + 2 * NP + lc, x);
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) x[c] *= sv.y;
+            f2 oc[CPL];
 #pragma unroll
             for (int k = 0; k < K4; ++k) {
               const ulonglong2 B = *reinterpret_cast<const ulonglong2*>(p + 64 * k + 4 * sub);
               const ulonglong2 C = *reinterpret_cast<const ulonglong2*>(p + NP + 64 * k + 4 * sub);
 #pragma unroll
-              for (int c = 0; c < SS_CPL; ++c) {
+              for (int c = 0; c < CPL; ++c) {
                 const f2 xd = pack_f2(x[c], x[c]);
                 S[c][2 * k] = fma_f2(kp, S[c][2 * k], fma_f2(am, S[c][2 * k], mul_f2(B.x, xd)));
                 S[c][2 * k + 1] = fma_f2(kp, S[c][2 * k + 1], fma_f2(am, S[c][2 * k + 1], mul_f2(B.y, xd)));
@@ -208,32 +200,32 @@ ssd_scan_kernel(SsdArgs a) {
               }
             }
 #pragma unroll
-            for (int c = 0; c < SS_CPL; ++c) {
+            for (int c = 0; c < CPL; ++c) {
               float lo, hi;
               unpack_f2(oc[c], lo, hi);
-              o[SS_CPL * tt + c] = lo + hi;
+              o[CPL * tt + c] = lo + hi;
             }
           }
         }
       }
-      // the run's 32 outputs of these four columns: lane `sub` gets those number 2 sub and 2 sub + 1
-      run_sums(o, lane);
-      const int tt = first + (sub >> 1), lcc = lc + (sub & 1) * 2, col = c0 + lcc;
+      // the run's outputs of these columns: lane `sub` gets CPL / 2 of token sub / 2's
+      run_sums<CPL>(o, lane);
+      const int tt = first + (sub >> 1), lcc = lc + (sub & 1) * (CPL / 2), col = c0 + lcc;
       if (tt < nt && col < P) {
-        const float2 x = *reinterpret_cast<const float2*>(sg + tt * PER_TOK + 2 * NP + lcc);
-        const float y0 = fmaf(skip, x.x, o[0]), y1 = fmaf(skip, x.y, o[1]);
+        const float* x = sg + tt * PER_TOK + 2 * NP + lcc;
         float* dst = a.out + (size_t)(base + tt) * inner + h * P + col;
-        if constexpr (VEC) {
-          *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+        if constexpr (VEC && CPL == 4) {
+          *reinterpret_cast<float2*>(dst) = make_float2(fmaf(skip, x[0], o[0]), fmaf(skip, x[1], o[1]));
         } else {
-          dst[0] = y0;
-          if (col + 1 < P) dst[1] = y1;
+#pragma unroll
+          for (int c = 0; c < CPL / 2; ++c)
+            if (col + c < P) dst[c] = fmaf(skip, x[c], o[c]);
         }
       }
     }
   }
 #pragma unroll
-  for (int c = 0; c < SS_CPL; ++c) {
+  for (int c = 0; c < CPL; ++c) {
     const int col = c0 + lc + c;
     if (col < P) store_column<K4, VEC>(st + (size_t)col * N, N, sub, S[c]);
   }
@@ -393,23 +385,27 @@ extern "C" int yalm_ssd_scan(const float* act, const float* dt, int dt_n, long l
     YALM_LAUNCH_CHECK();
     return 0;
   }
-  const dim3 grid((P + SS_COLS - 1) / SS_COLS, H, n_seqs), block(160);
-#define YALM_SSD1(K, V)                                                                                       \
+  const bool narrow = narrow_blocks((long long)((P + 31) / 32) * H * n_seqs);
+  const int cols = narrow ? 16 : 32;
+  const dim3 grid((P + cols - 1) / cols, H, n_seqs), block(160);
+#define YALM_SSD1(K, V, C)                                                                                    \
   do {                                                                                                        \
-    const size_t smem = (size_t)SS_STAGES * SS_TOK * (2 * 64 * K + SS_COLS) * sizeof(float);                  \
+    const size_t smem = (size_t)SS_STAGES * SS_TOK * (2 * 64 * K + 8 * C) * sizeof(float);                    \
     static bool set = false;                                                                                  \
     if (!set && smem > 40 * 1024) {                                                                           \
-      cudaError_t e = cudaFuncSetAttribute(ssd_scan_kernel<K, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaError_t e = cudaFuncSetAttribute(ssd_scan_kernel<K, V, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                            (int)smem);                                                        \
       if (e != cudaSuccess) return (int)e;                                                                    \
       set = true;                                                                                             \
     }                                                                                                         \
-    launch_pdl(ssd_scan_kernel<K, V>, grid, block, smem, stream, a);                                          \
+    launch_pdl(ssd_scan_kernel<K, V, C>, grid, block, smem, stream, a);                                       \
   } while (0)
-#define YALM_SSD(K)              \
-  do {                           \
-    if (vec) YALM_SSD1(K, true); \
-    else YALM_SSD1(K, false);    \
+#define YALM_SSD(K)                              \
+  do {                                           \
+    if (vec && narrow) YALM_SSD1(K, true, 2);    \
+    else if (vec) YALM_SSD1(K, true, 4);         \
+    else if (narrow) YALM_SSD1(K, false, 2);     \
+    else YALM_SSD1(K, false, 4);                 \
   } while (0)
   if (N <= 64) YALM_SSD(1);
   else if (N <= 128) YALM_SSD(2);

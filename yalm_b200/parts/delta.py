@@ -129,8 +129,7 @@ class GatedDeltaRule:
         if self.per_head:
             act = rt.buffer("delta_act", (n, ops.delta_head_row(H, G, dk, dv)), torch.float32)
             ops.short_conv(proj, S, 0, C, self.conv_w, view["conv"].state, batch, out32=act, silu=True)
-            ops.delta_prep(act, proj, S, self.col_b, 0, 0, None, H, G, dk, dv,
-                           head_decay=(self.col_a, self.dt_bias, self.a_log))
+            ops.delta_head_prep(act, proj, S, self.col_b, self.col_a, self.dt_bias, self.a_log, batch, H, G, dk, dv)
             o = rt.buffer("delta_o", (n, H * dv), torch.float32)
             ops.delta_head_scan(act, batch, view["state"].state, o, H, G, dk, dv)
             on = rt.buffer("delta_normed", (n, H * dv), rt.dtype)
