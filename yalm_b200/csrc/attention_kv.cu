@@ -8,8 +8,8 @@
 //    this step come from its own buffer, earlier ones from the cache.
 //  * attn_kv_decode (16-bit): one query per sequence, every key in the cache.  Transposed, S^T = K Q^T and
 //    O^T = V^T P^T: the 16 rows of a tile are keys (or features of a value) and its 8 columns the query heads
-//    that share a key head.  A warp walks through its own units of 16 keys with a cp.async ring of its own, so
-//    nothing but the end is a block's business; weights go from accumulators to operands in registers
+//    that share a key head.  A warp walks through its own units of 16 keys with two cp.async buffers of its own, so
+//    nothing but the end is a block's business, and two or three blocks share an SM; weights go from accumulators to operands in registers
 //    (movmatrix), three terms each.  Long sequences are split over blocks; the block that ends last merges.
 //  * attn_kv_fma: the same with 32-bit FMA on any storage type, any number of queries: the 32-bit path.
 //
@@ -299,7 +299,7 @@ attn_kv_prefill_kernel(KvArgs a) {
 }
 
 // ---- one query per sequence ---------------------------------------------------------------------------
-constexpr int KD_HEADS = 8, KD_KEYS = 16, KD_WARPS = 4, KD_STAGES = 3;
+constexpr int KD_HEADS = 8, KD_KEYS = 16, KD_WARPS = 4, KD_STAGES = 2;
 
 // NK, NV: 16-feature groups of keys and values (dk <= 16 NK, dv <= 16 NV).  grid (splits, G * tiles of 8 query
 // heads, sequences)
@@ -378,7 +378,7 @@ attn_kv_decode_kernel(KvArgs a) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) bias[e] = distance_bias(a, hd[e & 1], pos - (base + g + 8 * (e >> 1)));
     }
-    cp_wait<KD_STAGES - 2>();
+    cp_wait<KD_STAGES - 1>();
     __syncwarp();
     const T* ks = ring + (size_t)(u % KD_STAGES) * UNIT;
     const T* vs = ks + KD_KEYS * LDK;
