@@ -57,24 +57,38 @@ __global__ void __launch_bounds__(DP_THREADS) delta_head_prep_kernel(DeltaHeadPr
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int beta0 = 2 * a.G * a.dk + a.H * a.dv, hp = (a.H + 3) & ~3, tail = dh_tail(a.H, a.G, a.dk, a.dv);
   pdl_wait();
-  // 2 x 16 vectors over four warps: unit vectors, in memory and here
-  for (int i = warp; i < 2 * nt; i += DP_THREADS / 32) {
-    const int tt = i >> 1, is_k = i & 1;
-    float* v = a.act + (size_t)(t0 + tt) * a.row + (is_k * a.G + g) * a.dk;
-    float* d = (is_k ? k_s : q_s) + tt * pitch;
-    float x[8], ss = 0.f;                               // dk up to 256
+  // 2 x 16 vectors over four warps, four of a warp's at a time so that their loads are in flight together: unit
+  // vectors, in memory and here
+  constexpr int NW = DP_THREADS / 32, AT_ONCE = 4;
+  for (int i0 = warp; i0 < 2 * nt; i0 += NW * AT_ONCE) {
+    float x[AT_ONCE][8], ss[AT_ONCE];                   // dk up to 256
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int c = lane + 32 * j;
-      x[j] = c < a.dk ? v[c] : 0.f;
-      ss += x[j] * x[j];
+    for (int u = 0; u < AT_ONCE; ++u) {
+      const int i = i0 + u * NW, tt = i >> 1, is_k = i & 1;
+      const float* v = a.act + (size_t)(t0 + tt) * a.row + (is_k * a.G + g) * a.dk;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[u][j] = i < 2 * nt && lane + 32 * j < a.dk ? v[lane + 32 * j] : 0.f;
     }
-    const float r = (1.0f / sqrtf(warp_sum(ss) + 1e-6f)) * (is_k ? 1.0f : 1.0f / sqrtf((float)a.dk));
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int c = lane + 32 * j;
-      if (c < a.dk) v[c] = x[j] * r;
-      if (c < dkp) d[c] = x[j] * r;                     // zero beyond dk
+    for (int u = 0; u < AT_ONCE; ++u) {
+      ss[u] = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[u] += x[u][j] * x[u][j];
+      ss[u] = warp_sum(ss[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < AT_ONCE; ++u) {
+      const int i = i0 + u * NW, tt = i >> 1, is_k = i & 1;
+      if (i >= 2 * nt) continue;
+      float* v = a.act + (size_t)(t0 + tt) * a.row + (is_k * a.G + g) * a.dk;
+      float* d = (is_k ? k_s : q_s) + tt * pitch;
+      const float r = (1.0f / sqrtf(ss[u] + 1e-6f)) * (is_k ? 1.0f : 1.0f / sqrtf((float)a.dk));
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int c = lane + 32 * j;
+        if (c < a.dk) v[c] = x[u][j] * r;
+        if (c < dkp) d[c] = x[u][j] * r;                // zero beyond dk
+      }
     }
   }
   for (int i = threadIdx.x; i < nt * R; i += DP_THREADS) {
